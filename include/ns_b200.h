@@ -47,6 +47,9 @@ enum {
     NS_EPI_BIAS_RESIDUAL = 3 /* . + bias[n] + residual[m,n]      (x + Linear(...), Layers/Attention.cs:201-205) */
 };
 
+/* Activation of a gate. */
+enum { NS_ACT_SILU = 0, NS_ACT_SIGMOID = 1 };
+
 /* How a Linear layer is divided among tensor-parallel ranks. */
 enum { NS_SPLIT_NONE = 0, NS_SPLIT_COLUMN = 1, NS_SPLIT_ROW = 2 };
 
@@ -342,6 +345,10 @@ NS_API int ns_attention_prefill(ns_device_t dev, uint64_t q, uint64_t k, uint64_
  * forward yields a partial sum (see ns_bias_residual).  The reference has no counterpart for the split. */
 NS_API int ns_linear_create(ns_device_t dev, int K, int N, int mode, const float* w_kn, const float* bias, int split, int col_groups,
                             int tp_rank, int tp_size, ns_linear_t* linear);
+/* An NS_BF16 layer from bf16 weights [N, K] on the host (one row per output channel, as weight files of other frameworks store
+ * them), uploaded as they are; K and N are padded with zeros to multiples of 8 and ns_linear_info reports the padded sizes:
+ * the input rows are that long and padded with zeros.  No bias, no tensor-parallel split. */
+NS_API int ns_linear_create_bf16(ns_device_t dev, int N, int K, const void* w_nk, ns_linear_t* linear);
 NS_API int ns_linear_destroy(ns_linear_t linear);
 NS_API int ns_linear_info(ns_linear_t linear, int* k_local, int* n_local, int* mode, uint64_t* w, uint64_t* w_scale, uint64_t* bias);
 /* y[M, N_local] = epilogue(x . W^T).  NS_I8 layer: x int8 [M, K_local] with x_scale float [M] (from ns_quantize_rows_i8 or
@@ -362,9 +369,10 @@ NS_API int ns_linear_forward_host(ns_device_t dev, ns_linear_t linear, const flo
  * Fused row kernels of the decoding step.  With the few rows of a step, time goes to the NUMBER of launches; these
  * take over a product's epilogue so that the split-K second kernel and the row operator that follows are one launch.
  * ------------------------------------------------------------------------------------------------ */
-/* The int8 product of `linear` WITHOUT its epilogue: exact int32 partial sums [splits, M, N_local] are left in the device
- * object's scratch block (valid until the next call on this device that uses the scratch block: another product with a
- * split K, or decode attention with a split cache); `partial` and `splits` describe them.  M * N_local <= 2^24. */
+/* The product of `linear` WITHOUT its epilogue: exact int32 (NS_BF16 layer: float) partial sums [splits, M, N_local] are left
+ * in the device object's scratch block (valid until the next call on this device that uses the scratch block: another product
+ * with a split K, or decode attention with a split cache); `partial` and `splits` describe them.  M * N_local <= 2^24 (NS_BF16:
+ * 2^31). */
 NS_API int ns_linear_forward_partial(ns_device_t dev, ns_linear_t linear, uint64_t x, int M, uint64_t* partial, int* splits);
 /* x_out[m,n] = bf16(((float) sum_s partial[s,m,n] * x_scale[m]) * w_scale[n] + bias[n] + residual[m,n]) (residual bf16, may be
  * 0), then, when gamma != 0: q, q_scale = int8 row quantisation of bf16(LayerNorm(x_out)) -- the input of the next product.
@@ -398,6 +406,76 @@ NS_API int ns_linear_forward_norm_quant(ns_device_t dev, ns_linear_t linear, uin
 NS_API int ns_linear_forward_gelu_quant(ns_device_t dev, ns_linear_t linear, uint64_t x, uint64_t x_scale, int64_t rows, uint64_t q, uint64_t q_scale);
 NS_API int ns_linear_forward_kv_append(ns_device_t dev, ns_linear_t linear, uint64_t x, uint64_t x_scale, int batch, int steps, uint64_t qkv,
                                        ns_kv_cache_t cache, uint64_t page_table, int max_pages, uint64_t pos_dev);
+
+/* ------------------------------------------------------------------------------------------------
+ * Operators of decoders with a 32-bit residual stream, recurrent layers and latent attention.  No counterpart in the
+ * reference (LayerNorm, full attention and per-layer key/value caches only).
+ *
+ * A "source" is a product as its row kernel reads it: (address, splits, dtype, ld) = float partial sums [splits, rows, ld] that
+ * add up to the values (ns_linear_forward_partial), or one matrix [rows, ld] of NS_F32 / NS_BF16 with splits = 1.
+ * A "slot" is the place of a sequence in its model's state: `slots` (int32 [batch]) names the slot of every sequence of the
+ * step, `pos` and `last` (int32 [slot]) hold a slot's next position and last token (-1 before the first), and the caches and
+ * states are given as slot 0's address and the stride between slots in elements.  Rows are [batch, steps].
+ * Outputs that feed a product are written with a row pitch `*_ld` >= their width, padded with zeros.
+ * ------------------------------------------------------------------------------------------------ */
+/* y[b, i, :] = scale * table[token] + bigram[row], row = (previous token * mul_prev + token * mul_cur) mod buckets, and row
+ * `buckets` (the table's last) for a sequence's first token.  bigram may be 0.  Tables [rows, ld] of table_dtype, y float. */
+NS_API int ns_embed_ngram(ns_device_t dev, uint64_t ids, uint64_t table, int table_dtype, int table_ld, float scale, uint64_t bigram, int bigram_ld,
+                          int buckets, int64_t mul_prev, int64_t mul_cur, uint64_t slots, uint64_t last, int batch, int steps, int dim, int vocab, uint64_t y);
+/* x_out = x + alpha * source (float; x or the source may be 0; x_out may be 0 or x), then, when w != 0,
+ * y = x_out / sqrt(mean(x_out^2) + eps) * w of out_dtype.  row_map (int32 [rows], may be 0): output row r of y comes from row
+ * row_map[r]; src_rows is the number of rows of the source. */
+NS_API int ns_rms_rows(ns_device_t dev, uint64_t x, uint64_t src, int splits, int src_dtype, int src_ld, float alpha, uint64_t x_out, uint64_t w, float eps,
+                       uint64_t row_map, int64_t src_rows, int64_t rows, int cols, int out_dtype, uint64_t y, int y_ld);
+/* y[r, c] = gelu_tanh(source[r, c]) * source[r, ff + c] */
+NS_API int ns_glu_rows(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int64_t rows, int ff, int out_dtype, uint64_t y, int y_ld);
+/* y[r, 0:cols] = source[r, col:col+cols] in another type or pitch */
+NS_API int ns_copy_cols(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int col, int64_t rows, int cols, int out_dtype, uint64_t y,
+                        int y_ld);
+/* last[slot] = the step's last token of the sequence, pos[slot] += steps */
+NS_API int ns_seq_advance(ns_device_t dev, uint64_t ids, uint64_t slots, int batch, int steps, uint64_t pos, uint64_t last);
+/* int32 ids from the float-encoded ones of the sampler (ns_f32_sample_rows) */
+NS_API int ns_ids_from_f32(ns_device_t dev, uint64_t x, uint64_t ids, int n);
+
+/* Causal convolution over time per channel, then silu, then optionally every head made a unit vector
+ * (x / sqrt(sum x^2 + 1e-6)) times scales[s], for up to 4 tensors that lie side by side in the source.  fields: 9 int64 per
+ * tensor: first column, heads, channels per head, taps, unit (0 / 1), weight address (float [channels, taps], the current
+ * token's last), history address of slot 0 (float [taps, channels]: the raw inputs of earlier tokens at position modulo taps),
+ * output address ([rows, ld] of out_dtype), output ld.  The history of the step's sequences is read and replaced. */
+NS_API int ns_short_conv(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int segments, const int64_t* fields, const float* scales,
+                         int64_t hist_slot_stride, uint64_t slots, uint64_t pos, int batch, int steps, int out_dtype);
+/* Gated delta rule, token by token, in 32-bit floats: per head a state S [dim, vdim];
+ *   g = exp(-exp(a_log) * softplus(a + dt_bias)), beta = sigmoid(b);  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.
+ * q, k float [rows, kv_heads * dim] (head h uses q/k head h / (heads / kv_heads)), v and o float [rows, heads * vdim].
+ * per_channel 0: a at column a_col + head, dt_bias [heads]; 1: a at a_col + head * dim + channel, dt_bias [heads * dim].
+ * a and b are float sources; state float [heads, dim, vdim] per slot.  dim <= 256. */
+NS_API int ns_delta_recurrent(ns_device_t dev, uint64_t q, int q_ld, uint64_t k, int k_ld, uint64_t v, int v_ld, uint64_t a_src, int a_splits, int a_ld,
+                              int a_col, uint64_t b_src, int b_splits, int b_ld, int b_col, uint64_t a_log, uint64_t dt_bias, int per_channel,
+                              uint64_t state, int64_t state_slot_stride, uint64_t slots, int batch, int steps, int heads, int kv_heads, int dim, int vdim,
+                              uint64_t o, int o_ld);
+/* Per row and head: y = o / sqrt(mean(o^2) + eps) * w * act(gate), act NS_ACT_*; w float [vdim], gate at column gate_col of a
+ * source, y [rows, heads * vdim] of out_dtype. */
+NS_API int ns_gated_norm(ns_device_t dev, uint64_t o, int o_ld, uint64_t gate, int splits, int gate_dtype, int gate_ld, int gate_col, int act, uint64_t w,
+                         float eps, int64_t rows, int heads, int vdim, int out_dtype, uint64_t y, int y_ld);
+
+/* A row of the source is [query latent q_rank | latent kv_rank | rotated key part rot_dim].  cq = RMS norm of the first with
+ * q_norm; the cache row of the token's position (ring row = position modulo ring_len) = [RMS norm of the second with kv_norm |
+ * third with its first rot_dims entries, in neighbouring pairs, turned by position * freq[pair]].  cq and ring are of `dtype`. */
+NS_API int ns_latent_append(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int q_rank, int kv_rank, int rot_dim, int rot_dims,
+                            uint64_t q_norm, uint64_t kv_norm, float eps, uint64_t freq, uint64_t slots, uint64_t pos, int batch, int steps, int dtype,
+                            uint64_t cq, int cq_ld, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld);
+/* Heads laid out [dim | rot_dim]: the first part to plain[row * plain_ld + head * plain_head + c], the second, turned as above,
+ * to rot[row * rot_ld + head * rot_head + c]. */
+NS_API int ns_rotate_heads(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int heads, int dim, int rot_dim, int rot_dims, uint64_t freq,
+                           uint64_t slots, uint64_t pos, int batch, int steps, int plain_dtype, uint64_t plain, int64_t plain_ld, int plain_head,
+                           int rot_dtype, uint64_t rot, int64_t rot_ld, int rot_head);
+/* y[r * y_ld + head * y_head + n] = sum_k x[r * x_ld + head * x_head + k] * w[head * w_head + k * w_k + n * w_n], 32-bit sums. */
+NS_API int ns_head_matmul(ns_device_t dev, int x_dtype, uint64_t x, int64_t x_ld, int x_head, int w_dtype, uint64_t w, int64_t w_head, int64_t w_k, int64_t w_n,
+                          int y_dtype, uint64_t y, int64_t y_ld, int y_head, int rows, int heads, int k, int n);
+/* o[row, head, :] = softmax_j(scale * q[row, head, :] . ring[j, 0:width]) . ring[j, 0:rank] over positions j with
+ * 0 <= i - j < window (window 0: every earlier position); q float [rows, heads, width], o float [rows, heads, rank]. */
+NS_API int ns_latent_attend(ns_device_t dev, uint64_t q, int dtype, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld, int rank, int width,
+                            int window, float scale, uint64_t slots, uint64_t pos, int batch, int steps, int heads, uint64_t o);
 
 /* ------------------------------------------------------------------------------------------------
  * Tensor parallelism over NCCL.  No counterpart in the reference (single device; Device.cs:54-64).

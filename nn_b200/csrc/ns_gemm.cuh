@@ -41,8 +41,8 @@ struct NsGemmParams {
 // a: [M, K]; b: [N, K] (b_is_kn = false) or [K, N] (b_is_kn = true, bf16 only).
 // partial_override: when non-null, split-K partial sums go there (it must hold
 // k_splits * M * N 32-bit words) instead of the device object's scratch block.
-// deferred_partial / deferred_splits: when non-null (int8 kind only) the epilogue is left to a later kernel: exact
-// int32 partial sums [splits, M, N] stay in the device object's scratch block (one slab when K is not split) and the
+// deferred_partial / deferred_splits: when non-null the epilogue is left to a later kernel: exact int32 (bf16 kind:
+// float) partial sums [splits, M, N] stay in the device object's scratch block (one slab when K is not split) and the
 // two out-parameters describe them; no second kernel is launched.
 // tail: when non-null (int8 kind, [N, K] weights, M <= NS_TAIL_MAX_ROWS) the launch continues with the row operator
 // the struct describes (ns_tail.cuh).  For NS_TAIL_PEER the product writes its float partial rows to p.out (K is not

@@ -1066,7 +1066,6 @@ int ns_gemm_run(NsDevice* d, int kind, const void* a, const void* b, bool b_is_k
     int tail_splits = 0;
     if (tail != nullptr && !peer_tail) { deferred_partial = &tail_partial; deferred_splits = &tail_splits; }
     const bool deferred = deferred_partial != nullptr && deferred_splits != nullptr;
-    NS_REQUIRE(!deferred || kind == NS_KIND_I8, NS_ERR_ARGUMENT, "a deferred epilogue exists for int8 products only");
     const int elsize = kind == NS_KIND_I8 ? 1 : 2;
     NS_REQUIRE(M > 0 && N > 0 && K > 0, NS_ERR_ARGUMENT, "product with an empty dimension (M=%d N=%d K=%d)", M, N, K);
     NS_REQUIRE(((int64_t)K * elsize) % 16 == 0, NS_ERR_ARGUMENT, "K=%d: a row of %d bytes is not a multiple of 16 bytes", K, K * elsize);
@@ -1152,12 +1151,13 @@ int ns_gemm_run(NsDevice* d, int kind, const void* a, const void* b, bool b_is_k
             if (rc != NS_OK) return rc;
         }
     } else if (deferred) {
-        // K not split: the kernel writes its exact accumulators as the one slab and nothing else
+        // K not split: the kernel writes its accumulators (int8: exact int32, bf16: float) as the one slab and nothing else
         void* slab = nullptr;
         int rc = ns_scratch_reserve(d, (size_t)M * N * 4, &slab);
         if (rc != NS_OK) return rc;
-        p.raw = reinterpret_cast<int32_t*>(slab);
-        p.out = nullptr;
+        p.raw = kind == NS_KIND_I8 ? reinterpret_cast<int32_t*>(slab) : nullptr;
+        p.out = kind == NS_KIND_I8 ? nullptr : slab;
+        p.out_dtype = NS_F32;
         p.epilogue = NS_EPI_NONE;
     }
     CUtensorMap tmA, tmB;
@@ -1255,7 +1255,7 @@ int ns_gemm_run(NsDevice* d, int kind, const void* a, const void* b, bool b_is_k
     else rc = dispatch_bn<NS_KIND_BF16, true>(d, bn, tmA, tmB, sm, p);
     if (rc != NS_OK) return rc;
     if (deferred) {
-        *deferred_partial = p.k_splits > 1 ? p.partial : reinterpret_cast<void*>(p.raw);
+        *deferred_partial = p.k_splits > 1 ? p.partial : (kind == NS_KIND_I8 ? reinterpret_cast<void*>(p.raw) : p.out);
         *deferred_splits = p.k_splits;
         return NS_OK;
     }

@@ -101,6 +101,36 @@ extern "C" int ns_linear_create(ns_device_t h, int K, int N, int mode, const flo
     return NS_OK;
 }
 
+// A bf16 layer from weights that are bf16 already, one row per output channel: no conversion, no transpose.  Rows and columns
+// are padded with zeros to multiples of 8 (what TMA needs); the padded sizes are the layer's K and N.
+extern "C" int ns_linear_create_bf16(ns_device_t h, int N, int K, const void* w_nk, ns_linear_t* out)
+{
+    NsDevice* d = ns_dev(h);
+    int rc = ns_device_make_current(d);
+    if (rc != NS_OK) return rc;
+    NS_REQUIRE(out && w_nk && N > 0 && K > 0, NS_ERR_ARGUMENT, "ns_linear_create_bf16: bad argument");
+    NS_REQUIRE(!d->capturing, NS_ERR_STATE, "ns_linear_create_bf16: not allowed while the stream is being captured");
+    NsLinear* L = new NsLinear();
+    memset(L, 0, sizeof(*L));
+    L->ordinal = d->ordinal; L->mode = NS_BF16;
+    L->K = L->K_loc = (K + 7) / 8 * 8;
+    L->N = L->N_loc = (N + 7) / 8 * 8;
+    L->split = NS_SPLIT_NONE; L->tp_rank = 0; L->tp_size = 1;
+    const size_t pitch = (size_t)L->K * 2, bytes = pitch * L->N;
+    cudaError_t e = cudaMalloc(&L->w, bytes);
+    if (e == cudaSuccess && (L->K != K || L->N != N)) e = cudaMemsetAsync(L->w, 0, bytes, d->stream);
+    if (e == cudaSuccess) e = cudaMemcpy2DAsync(L->w, pitch, w_nk, (size_t)K * 2, (size_t)K * 2, N, cudaMemcpyHostToDevice, d->stream);
+    if (e == cudaSuccess) e = cudaStreamSynchronize(d->stream);
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        if (L->w) cudaFree(L->w);
+        delete L;
+        return ns_fail(NS_ERR_MEMORY, "ns_linear_create_bf16: %s (%d)", cudaGetErrorName(e), (int)e);
+    }
+    *out = reinterpret_cast<ns_linear_t>(L);
+    return NS_OK;
+}
+
 extern "C" int ns_linear_destroy(ns_linear_t lh)
 {
     NsLinear* L = reinterpret_cast<NsLinear*>(lh);
@@ -178,8 +208,8 @@ int ns_linear_forward_on(NsDevice* d, NsLinear* L, const void* x, const float* x
     return ns_gemm_run(d, L->mode == NS_I8 ? NS_KIND_I8 : NS_KIND_BF16, x, L->w, false, M, L->N_loc, L->K_loc, p);
 }
 
-// The int8 product of a layer without its epilogue: exact int32 partial sums [splits, M, N_local] stay in the device
-// object's scratch block for the row kernel that follows (ns_finish_norm_quant, ns_finish_kv_append).
+// The product of a layer without its epilogue: exact int32 (bf16 layers: float) partial sums [splits, M, N_local] stay in the
+// device object's scratch block for the row kernel that follows (ns_finish_norm_quant, ns_finish_kv_append; ns_rms_rows, ...).
 extern "C" int ns_linear_forward_partial(ns_device_t h, ns_linear_t lh, uint64_t x, int M, uint64_t* partial, int* splits)
 {
     NsDevice* d = ns_dev(h);
@@ -187,9 +217,9 @@ extern "C" int ns_linear_forward_partial(ns_device_t h, ns_linear_t lh, uint64_t
     if (rc != NS_OK) return rc;
     NsLinear* L = reinterpret_cast<NsLinear*>(lh);
     NS_REQUIRE(L && x && partial && splits, NS_ERR_ARGUMENT, "ns_linear_forward_partial: null argument");
-    NS_REQUIRE(L->mode == NS_I8, NS_ERR_ARGUMENT, "ns_linear_forward_partial: int8 layers only");
-    NS_REQUIRE(M > 0 && (int64_t)M * L->N_loc <= (int64_t)1 << 24, NS_ERR_ARGUMENT,
-               "ns_linear_forward_partial: meant for the few rows of a decoding step (M * N <= 2^24), got M=%d N=%d", M, L->N_loc);
+    const int64_t most = (int64_t)1 << (L->mode == NS_I8 ? 24 : 31);
+    NS_REQUIRE(M > 0 && (int64_t)M * L->N_loc <= most, NS_ERR_ARGUMENT,
+               "ns_linear_forward_partial: M=%d N=%d is more than the few rows of a decoding step", M, L->N_loc);
     NsGemmParams p = {};
     p.epilogue = NS_EPI_NONE;
     p.out_dtype = NS_F32;
@@ -197,7 +227,8 @@ extern "C" int ns_linear_forward_partial(ns_device_t h, ns_linear_t lh, uint64_t
     p.prefetch_b = 1;
     void* ptr = nullptr;
     int s = 0;
-    rc = ns_gemm_run(d, NS_KIND_I8, reinterpret_cast<const void*>(x), L->w, false, M, L->N_loc, L->K_loc, p, nullptr, 0, &ptr, &s);
+    rc = ns_gemm_run(d, L->mode == NS_I8 ? NS_KIND_I8 : NS_KIND_BF16, reinterpret_cast<const void*>(x), L->w, false, M, L->N_loc, L->K_loc, p, nullptr, 0,
+                     &ptr, &s);
     if (rc != NS_OK) return rc;
     *partial = reinterpret_cast<uint64_t>(ptr);
     *splits = s;

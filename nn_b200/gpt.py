@@ -24,6 +24,7 @@ from dataclasses import dataclass
 import numpy as np
 
 from . import native as N
+from .decoder import CachedDecoder
 from .device import Device, Storage
 
 
@@ -88,7 +89,7 @@ FLASH_MIN_STEPS = 128
 STREAM_MAX_ROWS = 16
 
 
-class GptW8A8:
+class GptW8A8(CachedDecoder):
     """weights: dict of float32 arrays in the reference's layouts --
     tok [V, D], pos [context, D], lnf_g, lnf_b [D], head_w [D, V], head_b [V], and per layer i:
     ln1_g, ln1_b, qkv_w [D, 3D], qkv_b, out_w [D, D], out_b, ln2_g, ln2_b, ff1_w [D, FF], ff1_b, ff2_w [FF, D], ff2_b
@@ -182,8 +183,7 @@ class GptW8A8:
         # Measured on the 24-layer model, batch 64: 2.49 ms per step against 2.44 with the row kernel of its own (the last
         # CTA of a row works alone while the others have left), so it stays off.
         self.attn_quant = False
-        self.graph = None
-        self.launches_per_step = 0
+        self.begin_decoding(cfg.context)
 
     # ------------------------------------------------------------------ one pass over `steps` new positions
     def _reduce_rows(self, lin: _Linear, m: int, x_in: Storage, x_out: Storage):
@@ -580,28 +580,6 @@ class GptW8A8:
         self._forward(t)
         self.length = t
 
-    def step(self, use_graph: bool = True) -> None:
-        """One cached decoding step for every sequence; the first call records it as a CUDA graph
-        (DecodingContext.CaptureStep / ReplayStep, Layers/Decoding.cs:129-155)."""
-        assert self.length + 1 <= self.cfg.context, "context is full: re-read the window first"
-        if not use_graph:
-            self._forward(1)
-        else:
-            if self.graph is None:
-                self._forward(1)               # un-captured once: sizes scratch memory, sets kernel attributes
-                self.length += 1
-                self.launches_per_step = self._n
-                self.dev.capture_begin()
-                try:
-                    self._forward(1)
-                except Exception:
-                    N.call("ns_capture_abort", self.dev.handle)
-                    raise
-                self.graph = self.dev.capture_end()
-                return                          # the captured pass did not execute; the un-captured one was this step
-            self.dev.graph_launch(self.graph)
-        self.length += 1
-
     def set_local_exchange(self, local: bool) -> None:
         """Measurement aid for several GPUs: with local=True the exchange kernel of the few-row pass runs in its
         single-rank form (this rank's own partial rows only: no flag traffic, no peer loads), so the step's time without
@@ -623,74 +601,8 @@ class GptW8A8:
             self.dev.graph_destroy(self.graph)
             self.graph = None
 
-    def read_ids(self) -> np.ndarray:
-        return self.ids.download(count=self.batch).copy()
-
     def read_logits(self) -> np.ndarray:
         return self.logits.download((self.batch, self.v_loc))
-
-    def generate(self, prompt: np.ndarray, n_new: int, use_graph: bool = True, marks: dict | None = None,
-                 mark_every: int = 32) -> tuple[np.ndarray, int]:
-        """Greedy decoding of n_new tokens per sequence; returns (tokens [batch, n_new], context resets).
-        marks: when a dict is given, device events are recorded into it on the device's stream -- "start" (before the
-        prompt is read), "prefill_end" (the first token is on the device), "steps" = [(tokens produced so far, event), ...]
-        every mark_every decoding steps and after the last one -- for timing a generation from outside."""
-        cfg, B = self.cfg, self.batch
-
-        def mark(name=None, count=None):
-            if marks is None:
-                return
-            e = self.dev.event()
-            self.dev.record(e)
-            if name is not None:
-                marks[name] = e
-            else:
-                marks.setdefault("steps", []).append((count, e))
-
-        history = [list(map(int, row)) for row in np.asarray(prompt)]
-        hist_dev = self.dev.empty(B * max(n_new, 1), N.NS_I32)
-        pending = 0            # tokens sampled on the device and not yet fetched
-        out: list[list[int]] = [[] for _ in range(B)]
-        resets = 0
-
-        def flush():
-            nonlocal pending
-            if pending:
-                got = hist_dev.download((pending, B), count=pending * B)
-                for row in got:
-                    for b in range(B):
-                        history[b].append(int(row[b])); out[b].append(int(row[b]))
-                pending = 0
-
-        def keep_token():
-            nonlocal pending
-            N.call("ns_d2d_async", self.dev.handle, C.c_uint64(hist_dev.ptr + pending * B * 4), C.c_uint64(self.ids.ptr), C.c_uint64(B * 4))
-            pending += 1
-
-        def window(keep):
-            return np.array([h[-keep:] for h in history], dtype=np.int32)
-
-        mark("start")
-        self.prefill(window(min(len(history[0]), cfg.context - 1)))
-        keep_token()
-        mark("prefill_end")
-        produced = 1
-        while produced < n_new:
-            if self.length >= cfg.context:
-                flush()
-                self.prefill(window(cfg.context // 2))     # window full: re-read the last half from position 0
-                keep_token()
-                resets += 1
-                produced += 1
-                continue
-            self.step(use_graph)
-            keep_token()
-            produced += 1
-            if (produced - 1) % mark_every == 0 or produced == n_new:
-                mark(count=produced)
-        flush()
-        self.dev.synchronize()
-        return np.array(out, dtype=np.int32)[:, :n_new], resets
 
     def close(self) -> None:
         if self.graph is not None:

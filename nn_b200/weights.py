@@ -131,3 +131,77 @@ def load_char_gpt(weights_path: str):
 def save_char_gpt(weights_path: str, cfg: GptConfig, w: dict, vocabulary: str) -> None:
     write_nsw2(weights_path, [w[name] for name, _ in gpt_tensor_names(cfg)])
     write_config(weights_path, cfg, vocabulary)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# model folders: config.json and model.safetensors
+# ---------------------------------------------------------------------------------------------------------------------
+_SAFETENSORS = {"BF16": np.dtype("<u2"), "F32": np.dtype("<f4"), "I32": np.dtype("<i4")}
+
+
+class SafeTensors:
+    """A safetensors file as a mapping name -> array, read tensor by tensor (the file stays mapped): little-endian u64 header
+    length, a JSON header name -> {dtype, shape, data_offsets}, then the data.  bf16 tensors come as their bits (uint16)."""
+
+    def __init__(self, path: str):
+        self.path = path
+        size = os.path.getsize(path)
+        with open(path, "rb") as f:
+            head = f.read(8)
+            n = struct.unpack("<Q", head)[0] if len(head) == 8 else size
+            if 8 + n > size:
+                raise InvalidDataError(f"{path} is not a safetensors file.")
+            try:
+                header = json.loads(f.read(n))
+            except ValueError:
+                raise InvalidDataError(f"{path}: the header is not JSON") from None
+        self._data = np.memmap(path, dtype=np.uint8, mode="r", offset=8 + n) if size > 8 + n else np.empty(0, np.uint8)
+        self.entries = {}
+        for name, e in header.items():
+            if name == "__metadata__":
+                continue
+            if e["dtype"] not in _SAFETENSORS:
+                raise InvalidDataError(f"{path}: {name} has type {e['dtype']}, which is not read here")
+            dt, (a, b) = _SAFETENSORS[e["dtype"]], e["data_offsets"]
+            if not 0 <= a <= b <= len(self._data) or b - a != int(np.prod(e["shape"], dtype=np.int64)) * dt.itemsize:
+                raise InvalidDataError(f"{path}: {name} does not fit the file")
+            self.entries[name] = (dt, tuple(e["shape"]), a, b)
+
+    def __contains__(self, name: str) -> bool:
+        return name in self.entries
+
+    def __iter__(self):
+        return iter(self.entries)
+
+    def shape(self, name: str) -> tuple:
+        return self.entries[name][1]
+
+    def __getitem__(self, name: str) -> np.ndarray:
+        dt, shape, a, b = self.entries[name]
+        return self._data[a:b].view(dt).reshape(shape) if a % dt.itemsize == 0 else np.frombuffer(self._data[a:b].tobytes(), dt).reshape(shape)
+
+
+def write_safetensors(path: str, tensors: dict) -> None:
+    """float32 and int32 arrays under their types, uint16 arrays as bf16 bits."""
+    names = {np.dtype(np.uint16): "BF16", np.dtype(np.float32): "F32", np.dtype(np.int32): "I32"}
+    header, at = {}, 0
+    for name, a in tensors.items():
+        n = int(a.nbytes)
+        header[name] = {"dtype": names[a.dtype], "shape": list(a.shape), "data_offsets": [at, at + n]}
+        at += n
+    text = json.dumps(header).encode()
+    text += b" " * (-len(text) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(text)) + text)
+        for a in tensors.values():
+            f.write(np.ascontiguousarray(a).tobytes())
+
+
+def check_shapes(tensors: SafeTensors, expected: dict) -> None:
+    """Every expected tensor is there in its shape (None: any size)."""
+    for name, shape in expected.items():
+        if name not in tensors:
+            raise InvalidDataError(f"{tensors.path}: tensor {name} is missing")
+        got = tensors.shape(name)
+        if len(got) != len(shape) or any(s is not None and s != g for s, g in zip(shape, got)):
+            raise InvalidDataError(f"Shape mismatch: file has {list(got)}, model has {list(shape)} ({name}).")
