@@ -840,6 +840,9 @@ def run_case(spec: str):
         print(json.dumps({"case": spec, "ok": True, "rows": m, "layer_us": total, "hbm_peak_gbs": peaks["hbm"], "ops": rows}))
         model.close()
         return
+    elif name == "fabezen":
+        print(json.dumps({"case": spec, "ok": True, **run_fabezen(dev, arg)}))
+        return
     elif name == "gpt_decode":
         from nn_b200 import dist as nsdist
         parts = arg.split(":") + ["", "", "", "", "", ""]
@@ -854,6 +857,149 @@ def run_case(spec: str):
         raise SystemExit(f"unknown case {spec}")
     dev.synchronize()
     print(json.dumps({"case": spec, "ok": True}))
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# Fabezen beside the int8 decoder at equal size
+# ---------------------------------------------------------------------------------------------------------------
+def fabezen_config(width: int, heads: int, ff: int, window: int, kinds: str, vocab: int = 32000, kv_rank: int = 512) -> dict:
+    """kinds: one letter per layer, d(elta), c(hannel-wise delta), l(atent attention); a kind's later layers use its first one's
+    tensors (the weights of three layers are more than L2 holds)."""
+    dim = width // heads
+    table = {"d": ("delta", {"heads": heads, "kv_heads": heads // 2, "dim": dim, "vdim": dim, "conv": 4}),
+             "c": ("channel_delta", {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4}),
+             "l": ("latent_attention", {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "q_rank": 3 * width // 4, "kv_rank": kv_rank,
+                                        "scale": (1.5 * dim) ** -0.5, "mask": {"size": window}, "rot": {"base": 10000.0, "dims": dim // 2}})}
+    layers, first = [], {}
+    for i, k in enumerate(kinds):
+        layer = {"type": table[k][0], "mixer": table[k][1], "mlp": {"kind": "dense", "ff": ff}}
+        if k in first:
+            layer["weights_of"] = first[k]
+        first.setdefault(k, i)
+        layers.append(layer)
+    return {"architecture": "Fabezen", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "embedding": {"scale": 8.0, "bigram": {"buckets": 32768, "mul_prev": 1009, "mul_cur": 31}}}
+
+
+class SyntheticFabezenWeights(dict):
+    """Random bf16 tensors made on first use; low ranks are the head size."""
+
+    def __init__(self, cfg: dict, low_rank: int):
+        from nn_b200.fabezen import FabezenConfig
+        super().__init__()
+        self.shapes = {k: tuple(low_rank if n is None else n for n in s) for k, s in FabezenConfig.from_dict(cfg).tensor_shapes().items()}
+
+    def __getitem__(self, key: str):
+        from nn_b200.blocks import bf16_bits
+        shape = self.shapes[key]
+        x = np.random.default_rng([11, zlib.crc32(key.encode())]).standard_normal(shape, dtype=np.float32)
+        last = key.rsplit(".", 1)[-1]
+        if last.startswith("norm"):
+            x = 1.0 + 0.1 * x
+        elif last in ("A_log", "dt_bias"):
+            x -= 2.0
+        elif key != "embed" and key != "bigram":
+            x *= shape[-1] ** -0.5
+        return bf16_bits(x)
+
+
+def fabezen_step_bytes(model, batch: int, context: int) -> float:
+    """Algorithmic HBM bytes of one decoding step: every product's weights, the recurrent states read and written, the cached rows
+    of the windows (bf16)."""
+    cfg, total = model.cfg, 2.0 * model.cfg.vocab * model.cfg.width
+    for layer in cfg.layers:
+        m, D = layer.mixer, cfg.width
+        if layer.type == "latent_attention":
+            H = m["heads"]
+            total += 2.0 * (m["q_rank"] * D + H * (m["dim"] + m["rot_dim"]) * m["q_rank"] + (m["kv_rank"] + m["rot_dim"]) * D + H * (m["dim"] + m["vdim"]) * m["kv_rank"]
+                            + D * H * m["vdim"])
+            total += 2.0 * batch * min(context, m["mask"]["size"]) * (m["kv_rank"] + m["rot_dim"])
+        else:
+            qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            total += 2.0 * D * (2 * qk + 2 * v + v) + 8.0 * batch * m["heads"] * m["dim"] * m["vdim"]
+        if layer.mlp:
+            total += 6.0 * D * layer.mlp["ff"]
+    return total
+
+
+def time_calls(dev, run, reps: int = 10, skip=("ns_h2d",)):
+    """Runs `run` once with every library call noted, then times each call alone: [(name, microseconds)] in order."""
+    from nn_b200 import native as N
+    calls, real = [], N.call
+
+    def noting(name, *args):
+        calls.append((name, args))
+        return real(name, *args)
+
+    N.call = noting
+    try:
+        run()
+    finally:
+        N.call = real
+    dev.synchronize()
+    e0, e1 = dev.event(), dev.event()
+    out = []
+    for name, args in calls:
+        if name in skip:
+            continue
+        real(name, *args)
+        dev.record(e0)
+        for _ in range(reps):
+            real(name, *args)
+        dev.record(e1)
+        out.append((name, dev.elapsed_ms(e0, e1) * 1e3 / reps))
+    return out
+
+
+def run_fabezen(dev, arg: str) -> dict:
+    """fabezen[:width:heads:ff:window:kinds:batch:prompt:new[:parts]] -- prefill and decoding throughput with random weights, and the
+    int8 decoder of equal width, heads, layers, batch and prompt beside it (its feed-forward has two matrices of 1.5 ff, as many
+    weights as the gated one's three).  `parts` instead times every library call of one prompt read and one step."""
+    from nn_b200.fabezen import Fabezen, FabezenConfig
+    from nn_b200.gpt import GptConfig, GptW8A8
+    f = (arg.split(":") if arg else []) + [""] * 9
+    width, heads, ff, window = int(f[0] or 2048), int(f[1] or 16), int(f[2] or 5632), int(f[3] or 512)
+    kinds, B, P, new = f[4] or "dcl", int(f[5] or 64), int(f[6] or 512), int(f[7] or 64)
+    peaks = measured_peaks()
+    cfg = fabezen_config(width, heads, ff, window, kinds)
+    model = Fabezen(dev, FabezenConfig.from_dict(cfg), SyntheticFabezenWeights(cfg, width // heads), batch=B, max_prefill=P)
+    prompt = np.random.default_rng(5).integers(0, cfg["vocab"], (B, P)).astype(np.int32)
+    if f[8] == "parts":
+        model.generate(prompt, 4)
+        dev.synchronize()
+        pre = time_calls(dev, lambda: model.prefill(prompt))
+        model.prefill(prompt)
+        model.step(False)
+        dec = time_calls(dev, lambda: model.step(False))
+        model.close()
+        return {"config": cfg["layers"], "batch": B, "prompt": P, "prefill_us": sum(t for _, t in pre), "decode_us": sum(t for _, t in dec),
+                "prefill": [[n, round(t, 1)] for n, t in pre], "decode": [[n, round(t, 1)] for n, t in dec]}
+
+    def timed(m):
+        m.generate(prompt, min(new, 8))
+        sampler = ClockSampler(dev.ordinal, "_fabezen")
+        sampler.start()
+        marks = {}
+        m.generate(prompt, new, marks=marks)
+        clocks = sampler.stop()
+        return {"prefill_ms": dev.elapsed_ms(marks["start"], marks["prefill_end"]), "ms_per_step": dev.elapsed_ms(marks["prefill_end"], marks["steps"][-1][1]) / (new - 1),
+                "launches_per_step": m.launches_per_step, "clocks": clocks}
+
+    rec = timed(model)
+    bytes_ = fabezen_step_bytes(model, B, P + new // 2)
+    model.close()
+    ctx = P + new
+    gcfg = GptConfig(vocab=cfg["vocab"], dim=width, heads=heads, layers=len(kinds), ff_dim=3 * ff // 2 // 256 * 256, context=ctx)
+    gpt = GptW8A8(dev, gcfg, SyntheticGptWeights(gcfg, 4), B, max_prefill=P)
+    ref = timed(gpt)
+    gpt.close()
+    gbytes = decode_step_bytes(gcfg, B, P + new / 2.0, 1)
+    for r, nbytes in ((rec, bytes_), (ref, gbytes)):
+        r["prefill_tokens_per_s"] = B * P / (r["prefill_ms"] * 1e-3)
+        r["decode_tokens_per_s"] = B / (r["ms_per_step"] * 1e-3)
+        r["decode_hbm_frac"] = nbytes / (r["ms_per_step"] * 1e-3) / 1e9 / peaks["hbm"]
+    return {"config": {"width": width, "heads": heads, "ff": ff, "window": window, "layers": kinds, "batch": B, "prompt": P, "new_tokens": new,
+                       "weights": "random, bf16", "peaks": peaks["source"]}, "fabezen": rec, "int8_gpt_equal_size": ref}
 
 
 def main():

@@ -49,7 +49,7 @@ def main(argv=None) -> int:
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="folder for the logits")
-    ap.add_argument("--max-tokens", type=int, default=0, help="most tokens that open sequences hold at a time")
+    ap.add_argument("--max-tokens", type=int, default=0, help="an upper bound of the tokens in open sequences (bounds the size of a pass)")
     args = ap.parse_args(argv)
     from .device import Device
     from .registry import load_model

@@ -40,12 +40,14 @@ def bigram_rows(tokens, buckets, mul_prev, mul_cur):
 def embedding(tokens, w, cfg):
     e = cfg["embedding"]
     x = w["embed"][np.asarray(tokens)] * e["scale"]
-    b = e["bigram"]
+    b = e.get("bigram")
+    if b is None:
+        return x
     return x + w["bigram"][bigram_rows(tokens, b["buckets"], b["mul_prev"], b["mul_cur"])]
 
 
 def short_conv(x, taps):
-    """x [T, channels], taps [channels, n] with the current token's weight last; zeros before the start; then silu."""
+    """x [T, channels], taps [channels, n]: column n - 1 weighs token t, column 0 token t - n + 1; the result goes through silu."""
     n = taps.shape[1]
     padded = np.concatenate([np.zeros((n - 1, x.shape[1])), x])
     return silu(sum(padded[j:j + len(x)] * taps[:, j] for j in range(n)))
@@ -112,7 +114,7 @@ def rotate(x, positions, base, dims):
 
 
 def windowed_softmax_attention(score, value, size):
-    """score [heads, T, T], value [T, heads, vdim]; position i sees j with 0 <= i - j < size."""
+    """score [heads, T, T], value [T, heads, vdim]; a query's own position and the size - 1 before it are visible."""
     T = score.shape[1]
     i, j = np.arange(T)[:, None], np.arange(T)[None, :]
     s = np.where((i >= j) & (i - j < size), score, -np.inf)
