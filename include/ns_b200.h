@@ -477,6 +477,20 @@ NS_API int ns_head_matmul(ns_device_t dev, int x_dtype, uint64_t x, int64_t x_ld
 NS_API int ns_latent_attend(ns_device_t dev, uint64_t q, int dtype, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld, int rank, int width,
                             int window, float scale, uint64_t slots, uint64_t pos, int batch, int steps, int heads, uint64_t o);
 
+/* The same on the tensor cores: q bf16 [rows, heads, width], ring bf16, o bf16 [rows, heads, rank]; meant for few tokens (all heads
+ * of a sequence share a cached row's read).  Uses the device object's scratch block when the window is split over CTAs. */
+NS_API int ns_latent_decode(ns_device_t dev, uint64_t q, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld, int rank, int width, int window,
+                            float scale, uint64_t slots, uint64_t pos, int batch, int steps, int heads, uint64_t o);
+/* keys[b, j, :] = the cached row (bf16) of position pos - past + j, j < rows; zeros before position 0. */
+NS_API int ns_latent_gather(ns_device_t dev, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld, int past, uint64_t slots, uint64_t pos, int batch,
+                            int rows, uint64_t keys);
+/* Windowed causal attention of a portion of `steps` tokens whose keys and values are expanded: q bf16 [rows, heads * (dim +
+ * rot_dim)] (rotated), kv bf16 [batch * (past + steps), heads * dim keys | heads * vdim values], keys as ns_latent_gather leaves
+ * them (the rotated key part, shared by all heads, at column rank), o bf16 [rows, heads * vdim]. */
+NS_API int ns_latent_prefill(ns_device_t dev, uint64_t q, int64_t q_ld, uint64_t kv, int64_t kv_ld, uint64_t keys, int64_t keys_ld, int rank, uint64_t slots,
+                             uint64_t pos, int batch, int steps, int heads, int dim, int rot_dim, int vdim, int past, int window, float scale, uint64_t o,
+                             int64_t o_ld);
+
 /* ------------------------------------------------------------------------------------------------
  * Tensor parallelism over NCCL.  No counterpart in the reference (single device; Device.cs:54-64).
  * ------------------------------------------------------------------------------------------------ */

@@ -44,19 +44,20 @@ class Workspace:
 
     def __init__(self, dev: Device, dtype: int):
         self.dev, self.dtype = dev, dtype
-        self._need: dict[str, tuple[int, int]] = {}
+        self._need: dict[str, tuple[int, set]] = {}
         self._buf: dict[str, object] = {}
 
-    def need(self, name: str, per_row: int, dtype: int | None = None) -> None:
+    def need(self, name: str, per_row: int, dtype: int | None = None, extra: int = 0) -> None:
+        """per_row elements for each of a pass's rows, and for `extra` more rows per sequence."""
         dtype = self.dtype if dtype is None else dtype
-        have = self._need.get(name, (0, dtype))
-        assert have[1] == dtype
-        self._need[name] = (max(have[0], per_row), dtype)
+        have = self._need.setdefault(name, (dtype, set()))
+        assert have[0] == dtype
+        have[1].add((per_row, extra))
 
-    def allocate(self, rows: int) -> None:
+    def allocate(self, rows: int, batch: int) -> None:
         self.rows = rows
-        for name, (per_row, dtype) in self._need.items():
-            self._buf[name] = self.dev.zeros(rows * per_row, dtype)
+        for name, (dtype, sizes) in self._need.items():
+            self._buf[name] = self.dev.zeros(max(per_row * (rows + batch * extra) for per_row, extra in sizes), dtype)
 
     def __getitem__(self, name: str) -> int:
         return self._buf[name].ptr
@@ -69,6 +70,7 @@ class Step:
     steps: int
     slots: int
     pos: int
+    longest: int = 0         # the most tokens one of the sequences has behind it
     launches: int = 0
 
     @property
@@ -134,13 +136,14 @@ class Product:
         step.launches += 1
         return Source(ptr.value, splits.value, N.NS_F32, self.ld)
 
-    def into(self, x: int, m: int, y: int) -> None:
-        """Float output [m, ld] at y."""
+    def into(self, x: int, m: int, y: int, dtype: int = N.NS_F32) -> None:
+        """Output [m, ld] at y (bf16 layers: of either type)."""
         if self.handle is None:
+            assert dtype == N.NS_F32
             N.call("ns_f32_batched_matmul", self.dev.handle, C.c_uint64(x), C.c_uint64(self.w_ptr), C.c_uint64(y), 1, m, self.ld, self.k_ld, 0, 1,
                    C.c_float(0.0))
         else:
-            N.call("ns_linear_forward", self.dev.handle, self.handle, C.c_uint64(x), C.c_uint64(0), m, N.EPI_NONE, C.c_uint64(0), N.NS_F32, N.NS_F32,
+            N.call("ns_linear_forward", self.dev.handle, self.handle, C.c_uint64(x), C.c_uint64(0), m, N.EPI_NONE, C.c_uint64(0), N.NS_F32, dtype,
                    C.c_uint64(y))
 
     def close(self) -> None:
@@ -261,9 +264,16 @@ class DeltaMixer:
 
 
 class LatentAttentionMixer:
-    """Attention over cached latents with a sliding window (ns_latent.cu).
+    """Attention over cached latents with a sliding window (ns_latent.cu, ns_latent_tc.cu).
 
-    weights: dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o."""
+    weights: dq, dq_norm, uq, dkv, dkv_norm, uk, uv, o.
+
+    Two forms of the same attention.  Few tokens: the unrotated query goes through its head's key matrix, attention runs over the
+    cached latents as one key / value head shared by all, the weighted latent goes through the head's value matrix.  A prompt's
+    portion (bf16): keys and values of the window are expanded by one product and attention runs per head.  The choice depends on
+    the portion's length alone, so a sequence goes through the same arithmetic in any batch."""
+
+    EXPAND_STEPS = 32        # portions of at least this many tokens are expanded
 
     def __init__(self, ws: Workspace, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, window: int, rot_base: float,
                  rot_dims: int, eps: float, w: dict):
@@ -276,13 +286,18 @@ class LatentAttentionMixer:
         self.freq = dev.from_numpy((float(rot_base) ** (-2.0 * i / max(rot_dims, 1))).astype(np.float32))
         self.down = Product(ws, w["dq"], w["dkv"])
         self.uq = Product(ws, w["uq"])
+        # its input rows are whole cached rows: the columns of the rotated part are zero
+        self.kv = Product(ws, *(np.pad(w[n], ((0, 0), (0, rot_dim))) for n in ("uk", "uv")))
         self.out = Product(ws, w["o"])
-        per_head = (lambda a: dev.from_numpy(bf16_bits(a).reshape(-1))) if ws.dtype == N.NS_BF16 else (lambda a: dev.from_numpy(f32(a).reshape(-1)))
-        self.uk, self.uv = per_head(w["uk"]), per_head(w["uv"])
+        self.expands = ws.dtype == N.NS_BF16 and vdim <= 256 and dim + rot_dim <= 512
         ws.need("cq", self.uq.k_ld)
         ws.need("plain", heads * dim)
-        ws.need("carried", heads * self.width, N.NS_F32)
-        ws.need("weighted", heads * kv_rank, N.NS_F32)
+        ws.need("carried", heads * self.width)
+        ws.need("weighted", heads * kv_rank)
+        if self.expands:
+            ws.need("q_heads", heads * (dim + rot_dim))
+            ws.need("keys", pad8(self.width), extra=window - 1)
+            ws.need("kv", self.kv.ld, extra=window - 1)
         # the columns that pad a row of the output product's input are never written: a buffer of this width's own keeps them zero
         self.mixed = f"mixed_{heads * vdim}"
         ws.need(self.mixed, self.out.k_ld)
@@ -296,23 +311,38 @@ class LatentAttentionMixer:
         u, i64 = C.c_uint64, C.c_int64
         ring: Reservation = cache["ring"]
         at = (u(step.slots), u(step.pos), step.batch, step.steps)
+        ring_args = (u(ring.ptr), i64(ring.stride), cache["len"], pad8(W))
         s = self.down(h, step)
         N.call("ns_latent_append", hd, *s.args, self.q_rank, R, self.rot_dim, self.rot_dims, u(self.q_norm.ptr), u(self.kv_norm.ptr), C.c_float(self.eps),
-               u(self.freq.ptr), *at, dt, u(ws["cq"]), self.uq.k_ld, u(ring.ptr), i64(ring.stride), cache["len"], pad8(W))
+               u(self.freq.ptr), *at, dt, u(ws["cq"]), self.uq.k_ld, *ring_args)
         s = self.uq(ws["cq"], step)
-        carried = ws["carried"]
-        N.call("ns_rotate_heads", hd, *s.args, H, self.dim, self.rot_dim, self.rot_dims, u(self.freq.ptr), *at, dt, u(ws["plain"]), i64(H * self.dim), self.dim,
-               N.NS_F32, u(carried + 4 * R), i64(H * W), W)
+        rotate = (hd, *s.args, H, self.dim, self.rot_dim, self.rot_dims, u(self.freq.ptr), *at)
+        mixed = ws[self.mixed]
+        if self.expands and step.steps >= self.EXPAND_STEPS:
+            qw = self.dim + self.rot_dim
+            q, past = ws["q_heads"], min(self.window - 1, step.longest)
+            N.call("ns_rotate_heads", *rotate, dt, u(q), i64(H * qw), qw, dt, u(q + 2 * self.dim), i64(H * qw), qw)
+            N.call("ns_latent_gather", hd, *ring_args, past, u(step.slots), u(step.pos), step.batch, past + step.steps, u(ws["keys"]))
+            self.kv.into(ws["keys"], step.batch * (past + step.steps), ws["kv"], dt)
+            N.call("ns_latent_prefill", hd, u(q), i64(H * qw), u(ws["kv"]), i64(self.kv.ld), u(ws["keys"]), i64(pad8(W)), R, *at, H, self.dim, self.rot_dim,
+                   self.vdim, past, self.window, C.c_float(self.scale), u(mixed), i64(self.out.k_ld))
+            step.launches += 5
+            return self.out(mixed, step)
+        el, carried, k_ld = _SIZE[dt], ws["carried"], self.kv.k_ld
+        N.call("ns_rotate_heads", *rotate, dt, u(ws["plain"]), i64(H * self.dim), self.dim, dt, u(carried + el * R), i64(H * W), W)
         # the unrotated query through the head's key matrix: its score with a latent is then one dot product
-        N.call("ns_head_matmul", hd, dt, u(ws["plain"]), i64(H * self.dim), self.dim, dt, u(self.uk.ptr), i64(self.dim * R), i64(R), i64(1), N.NS_F32,
+        N.call("ns_head_matmul", hd, dt, u(ws["plain"]), i64(H * self.dim), self.dim, dt, u(self.kv.w_ptr), i64(self.dim * k_ld), i64(k_ld), i64(1), dt,
                u(carried), i64(H * W), W, step.m, H, self.dim, R)
-        N.call("ns_latent_attend", hd, u(carried), dt, u(ring.ptr), i64(ring.stride), cache["len"], pad8(W), R, W, self.window, C.c_float(self.scale), *at, H,
-               u(ws["weighted"]))
-        N.call("ns_head_matmul", hd, N.NS_F32, u(ws["weighted"]), i64(H * R), R, dt, u(self.uv.ptr), i64(self.vdim * R), i64(1), i64(R), dt, u(ws[self.mixed]),
-               i64(self.out.k_ld), self.vdim, step.m, H, R, self.vdim)
+        attend = (*ring_args, R, W, self.window, C.c_float(self.scale), *at, H, u(ws["weighted"]))
+        if dt == N.NS_BF16:
+            N.call("ns_latent_decode", hd, u(carried), *attend)
+        else:
+            N.call("ns_latent_attend", hd, u(carried), dt, *attend)
+        N.call("ns_head_matmul", hd, dt, u(ws["weighted"]), i64(H * R), R, dt, u(self.kv.w_ptr + el * H * self.dim * k_ld), i64(self.vdim * k_ld), i64(1), i64(k_ld),
+               dt, u(mixed), i64(self.out.k_ld), self.vdim, step.m, H, R, self.vdim)
         step.launches += 5
-        return self.out(ws[self.mixed], step)
+        return self.out(mixed, step)
 
     def close(self) -> None:
-        for p in (self.down, self.uq, self.out):
+        for p in (self.down, self.uq, self.kv, self.out):
             p.close()

@@ -10,6 +10,9 @@
 // no counterpart.
 #include "ns_seq.cuh"
 
+int ns_head_matmul_tc(NsDevice* d, uint64_t x, int64_t x_ld, int x_head, uint64_t w, int64_t w_head, int64_t w_k, int64_t w_n, int y_dtype, uint64_t y, int64_t y_ld,
+                      int y_head, int rows, int heads, int k, int n);   // ns_latent_tc.cu
+
 namespace {
 
 // ---------------------------------------------------------------------------------------------
@@ -335,6 +338,8 @@ extern "C" int ns_head_matmul(ns_device_t h, int x_dtype, uint64_t x, int64_t x_
     NS_REQUIRE(x && w && y && rows > 0 && heads > 0 && k > 0 && n > 0, NS_ERR_ARGUMENT, "ns_head_matmul: bad argument");
     NS_REQUIRE(float_or_bf16(x_dtype) && float_or_bf16(w_dtype) && float_or_bf16(y_dtype), NS_ERR_ARGUMENT, "ns_head_matmul: bad types");
     NS_REQUIRE(heads <= 65535 && (rows + 63) / 64 <= 65535, NS_ERR_ARGUMENT, "ns_head_matmul: too many rows or heads");
+    if (x_dtype == NS_BF16 && w_dtype == NS_BF16 && (w_k == 1 || w_n == 1))
+        return ns_head_matmul_tc(d, x, x_ld, x_head, w, w_head, w_k, w_n, y_dtype, y, y_ld, y_head, rows, heads, k, n);
     HeadMatmulArgs a;
     a.x = reinterpret_cast<const void*>(x); a.x_ld = x_ld; a.x_head = x_head;
     a.w = reinterpret_cast<const void*>(w); a.w_head = w_head; a.w_k = w_k; a.w_n = w_n;
@@ -346,7 +351,6 @@ extern "C" int ns_head_matmul(ns_device_t h, int x_dtype, uint64_t x, int64_t x_
         return NS_OK;
     };
     if (x_dtype == NS_F32 && w_dtype == NS_F32 && y_dtype == NS_F32) return go(ns_head_matmul_kernel<float, float, float>);
-    if (x_dtype == NS_BF16 && w_dtype == NS_BF16 && y_dtype == NS_F32) return go(ns_head_matmul_kernel<uint16_t, uint16_t, float>);
     if (x_dtype == NS_F32 && w_dtype == NS_BF16 && y_dtype == NS_BF16) return go(ns_head_matmul_kernel<float, uint16_t, uint16_t>);
     if (x_dtype == NS_F32 && w_dtype == NS_BF16 && y_dtype == NS_F32) return go(ns_head_matmul_kernel<float, uint16_t, float>);
     return ns_fail(NS_ERR_ARGUMENT, "ns_head_matmul: this combination of types is not built");

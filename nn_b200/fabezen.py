@@ -157,7 +157,7 @@ class Fabezen(CachedDecoder):
         ws.need("h", pad8(D))
         rows = batch * max_prefill
         self.logit_rows = max(batch, self.LOGIT_ROWS)
-        ws.allocate(max(rows, self.logit_rows))
+        ws.allocate(max(rows, self.logit_rows), batch)
         self.states.allocate()
         self.logits_padded = dev.empty(self.logit_rows * self.head.ld, N.NS_F32)
         self.logits = self.logits_padded if self.head.ld == cfg.vocab else dev.empty(self.logit_rows * cfg.vocab, N.NS_F32)
@@ -206,9 +206,9 @@ class Fabezen(CachedDecoder):
                C.c_uint64(self.states.pos.ptr), C.c_uint64(self.states.last.ptr))
         step.launches += 1
 
-    def _step(self, batch: int, steps: int) -> Step:
+    def _step(self, batch: int, steps: int, longest: int) -> Step:
         assert batch * steps <= self.ws.rows and steps <= self.max_prefill
-        return Step(batch, steps, self.slot_ids.ptr, self.states.pos.ptr)
+        return Step(batch, steps, self.slot_ids.ptr, self.states.pos.ptr, longest)
 
     def _use_slots(self, slots: list[int]) -> None:
         if slots != self._slots_now:
@@ -238,7 +238,7 @@ class Fabezen(CachedDecoder):
         for at in range(0, t, self.max_prefill):
             n = min(self.max_prefill, t - at)
             self._put(self.ids, ids[:, at:at + n])
-            step = self._step(b, n)
+            step = self._step(b, n, max(self.states.position[s] for s in slots) + at)
             self._layers(step)
             self._advance(step)
             here = [i for i, (_, p) in enumerate(pairs) if at <= p < at + n]
@@ -259,7 +259,7 @@ class Fabezen(CachedDecoder):
         self.drop_graph()
 
     def _forward(self, steps: int) -> None:
-        step = self._step(self.batch, steps)
+        step = self._step(self.batch, steps, self.length)
         self._layers(step)
         self._advance(step)
         self._head(step, self.batch)
@@ -282,16 +282,17 @@ class Fabezen(CachedDecoder):
         if self._lockstep is None:
             self._lockstep = [self.states.open() for _ in range(b)]
         else:
-            for s in self._lockstep:
-                self.states.rewind(s)
+            self.states.rewind(*self._lockstep)
         self._use_slots(self._lockstep)
+        self.length = 0
         for at in range(0, t, self.max_prefill):
             n = min(self.max_prefill, t - at)
             self._put(self.ids, ids[:, at:at + n])
             if at + n < t:
-                step = self._step(b, n)
+                step = self._step(b, n, at)
                 self._layers(step)
                 self._advance(step)
+                self.length += n
             else:
                 self._last_rows(n)
                 self._forward(n)

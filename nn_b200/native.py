@@ -104,6 +104,9 @@ SIGNATURES = {
     "ns_rotate_heads": [vp, u64, i32, i32, i32, i32, i32, i32, i32, u64, u64, u64, i32, i32, i32, u64, i64, i32, i32, u64, i64, i32],
     "ns_head_matmul": [vp, i32, u64, i64, i32, i32, u64, i64, i64, i64, i32, u64, i64, i32, i32, i32, i32, i32],
     "ns_latent_attend": [vp, u64, i32, u64, i64, i32, i32, i32, i32, i32, f32, u64, u64, i32, i32, i32, u64],
+    "ns_latent_decode": [vp, u64, u64, i64, i32, i32, i32, i32, i32, f32, u64, u64, i32, i32, i32, u64],
+    "ns_latent_gather": [vp, u64, i64, i32, i32, i32, u64, u64, i32, i32, u64],
+    "ns_latent_prefill": [vp, u64, i64, u64, i64, u64, i64, i32, u64, u64, i32, i32, i32, i32, i32, i32, i32, i32, f32, u64, i64],
     "ns_bias_residual": [vp, u64, u64, u64, i32, i64, i32, i32, u64],
     "ns_argmax_partial": [vp, u64, i32, i32, i64, i32, u64, u64],
     "ns_argmax_merge": [vp, u64, u64, i32, i32, u64],

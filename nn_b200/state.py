@@ -63,13 +63,22 @@ class SequenceStates:
         self.rewind(slot)
         return slot
 
-    def rewind(self, slot: int) -> None:
-        h = self.dev.handle
-        if self._bytes[0]:
-            N.call("ns_memset32_async", h, C.c_uint64(self.blocks[0].ptr + slot * self._bytes[0]), 0, C.c_uint64(self._bytes[0] // 4))
-        N.call("ns_memset32_async", h, C.c_uint64(self.pos.ptr + 4 * slot), 0, C.c_uint64(1))
-        N.call("ns_memset32_async", h, C.c_uint64(self.last.ptr + 4 * slot), 0xFFFFFFFF, C.c_uint64(1))
-        self.position[slot] = 0
+    def rewind(self, *slots: int) -> None:
+        """Back to position 0, everything cleared; neighbouring slots are cleared together."""
+        h, order = self.dev.handle, sorted(slots)
+        at = 0
+        while at < len(order):
+            n = 1
+            while at + n < len(order) and order[at + n] == order[at] + n:
+                n += 1
+            first = order[at]
+            if self._bytes[0]:
+                N.call("ns_memset32_async", h, C.c_uint64(self.blocks[0].ptr + first * self._bytes[0]), 0, C.c_uint64(n * self._bytes[0] // 4))
+            N.call("ns_memset32_async", h, C.c_uint64(self.pos.ptr + 4 * first), 0, C.c_uint64(n))
+            N.call("ns_memset32_async", h, C.c_uint64(self.last.ptr + 4 * first), 0xFFFFFFFF, C.c_uint64(n))
+            at += n
+        for s in slots:
+            self.position[s] = 0
 
     def close(self, slot: int) -> None:
         del self.position[slot]

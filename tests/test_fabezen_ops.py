@@ -300,8 +300,12 @@ def test_head_products(dev, rows, H, k, n, transposed):
         close(got, want if xd == N.NS_F32 else want_b, 2e-5 if yd == N.NS_F32 else 3e-2)
 
 
-def attend(dev, q, ring_rows, window, pos, steps, rank, scale, dtype, ring_len):
+FORMS = {"f32": N.NS_F32, "f32_on_bf16_rows": N.NS_BF16, "tensor_cores": N.NS_BF16}
+
+
+def attend(dev, q, ring_rows, window, pos, steps, rank, scale, form, ring_len):
     """q [B, steps, H, width]; ring_rows [B, pos + steps, width] by position."""
+    dtype = FORMS[form]
     B, _, H, width = q.shape
     ld = (width + 7) // 8 * 8
     st = Slots(dev, list(range(B)), [pos] * B)
@@ -309,9 +313,14 @@ def attend(dev, q, ring_rows, window, pos, steps, rank, scale, dtype, ring_len):
     for p in range(max(0, pos + steps - ring_len), pos + steps):
         ring[:, p % ring_len, :width] = ring_rows[:, p]
     dr = dev.from_numpy(ring if dtype == N.NS_F32 else bf16_bits(ring))
+    tail = (u(dr.ptr), i64(ring_len * ld), ring_len, ld, rank, width, window, fl(scale), u(st.slots.ptr), u(st.pos.ptr), B, steps, H)
+    if form == "tensor_cores":
+        dq, o = dev.from_numpy(bf16_bits(q)), dev.empty(B * steps * H * rank, N.NS_BF16)
+        N.call("ns_latent_decode", dev.handle, u(dq.ptr), *tail, u(o.ptr))
+        dev.synchronize()
+        return f32(o.download((B, steps, H, rank)))
     dq, o = dev.from_numpy(q.astype(np.float32)), dev.empty(B * steps * H * rank)
-    N.call("ns_latent_attend", dev.handle, u(dq.ptr), dtype, u(dr.ptr), i64(ring_len * ld), ring_len, ld, rank, width, window, fl(scale), u(st.slots.ptr),
-           u(st.pos.ptr), B, steps, H, u(o.ptr))
+    N.call("ns_latent_attend", dev.handle, u(dq.ptr), dtype, *tail, u(o.ptr))
     dev.synchronize()
     return o.download((B, steps, H, rank))
 
@@ -329,22 +338,22 @@ def attend_oracle(q, rows, window, pos, rank, scale):
     return out
 
 
-@pytest.mark.parametrize("dtype", [N.NS_F32, N.NS_BF16])
+@pytest.mark.parametrize("form", list(FORMS))
 @pytest.mark.parametrize("H,rank,rd,window,pos,steps", [(1, 16, 2, 1, 0, 1), (3, 44, 12, 11, 5, 9), (9, 136, 16, 70, 300, 3), (16, 512, 64, 129, 1000, 2),
-                                                       (5, 64, 8, 33, 31, 1), (5, 64, 8, 64, 0, 130)])
-def test_latent_attention_over_the_ring(dev, dtype, H, rank, rd, window, pos, steps):
+                                                       (5, 64, 8, 33, 31, 1), (5, 64, 8, 64, 0, 130), (40, 256, 32, 1000, 2000, 1), (2, 700, 20, 200, 90, 4)])
+def test_latent_attention_over_the_ring(dev, form, H, rank, rd, window, pos, steps):
     rng = rng_for(10, H, rank, window)
     width = rank + rd
     rows = f32(bf16_bits(rng.standard_normal((2, pos + steps, width))))
-    q = rng.standard_normal((2, steps, H, width)).astype(np.float32)
+    q = f32(bf16_bits(rng.standard_normal((2, steps, H, width))))
     scale = 1.5 / np.sqrt(width)
-    got = attend(dev, q, rows, window, pos, steps, rank, scale, dtype, window - 1 + steps + 2)
-    close(got, attend_oracle(q.astype(np.float64), rows.astype(np.float64), window, pos, rank, scale), 3e-5 if dtype == N.NS_F32 else 2e-3)
+    got = attend(dev, q, rows, window, pos, steps, rank, scale, form, window - 1 + steps + 2)
+    close(got, attend_oracle(q.astype(np.float64), rows.astype(np.float64), window, pos, rank, scale), 3e-2 if form == "tensor_cores" else 3e-5)
 
 
-@pytest.mark.parametrize("dtype", [N.NS_F32, N.NS_BF16])
+@pytest.mark.parametrize("form", list(FORMS))
 @pytest.mark.parametrize("window", [1, 2, 31, 32, 33, 64, 65, 100])
-def test_a_standing_out_key_at_the_windows_edges(dev, dtype, window):
+def test_a_standing_out_key_at_the_windows_edges(dev, form, window):
     """One key takes nearly all weight where it is seen, and none one token further."""
     H, rank, rd, pos, steps = 2, 32, 8, 150, 3
     width = rank + rd
@@ -358,5 +367,50 @@ def test_a_standing_out_key_at_the_windows_edges(dev, dtype, window):
             j = pos + i - back
             rows = base.copy()
             rows[0, j, 0], rows[0, j, 1] = 30.0, 16.0
-            got = attend(dev, q, rows, window, pos, steps, rank, 1.0, dtype, window - 1 + steps)[0, i]
+            got = attend(dev, q, rows, window, pos, steps, rank, 1.0, form, window - 1 + steps)[0, i]
             assert (abs(got[:, 1] - 16.0).max() < 0.05) if seen else (abs(got[:, 1]).max() < 1.0), (i, back)
+
+
+@pytest.mark.parametrize("H,dim,rd,vdim,rank,window,pos,steps", [(2, 16, 2, 16, 16, 1, 0, 5), (3, 20, 12, 36, 44, 11, 0, 40), (3, 20, 12, 36, 44, 70, 31, 64),
+                                                                (4, 48, 16, 80, 136, 65, 500, 130), (2, 128, 64, 128, 512, 128, 40, 200), (1, 64, 32, 200, 64, 300, 7, 65)])
+def test_expanded_attention_of_a_portion(dev, H, dim, rd, vdim, rank, window, pos, steps):
+    rng = rng_for(12, H, dim, window, steps)
+    B, ld = 2, (rank + rd + 7) // 8 * 8
+    poss = [pos, max(0, pos - 3)]
+    past = min(window - 1, max(poss))
+    ring_len = window - 1 + steps
+    cached = f32(bf16_bits(rng.standard_normal((B, max(poss) + steps, rank + rd))))
+    ring = np.full((B, ring_len, ld), 5.0, np.float32)
+    for b in range(B):
+        for p in range(max(0, poss[b] + steps - ring_len), poss[b] + steps):
+            ring[b, p % ring_len] = 0.0
+            ring[b, p % ring_len, :rank + rd] = cached[b, p]
+    st, dr, keys = Slots(dev, [0, 1], poss), dev.from_numpy(bf16_bits(ring)), dev.empty(B * (past + steps) * ld, N.NS_BF16)
+    nk = past + steps
+    N.call("ns_latent_gather", dev.handle, u(dr.ptr), i64(ring_len * ld), ring_len, ld, past, u(st.slots.ptr), u(st.pos.ptr), B, nk, u(keys.ptr))
+    dev.synchronize()
+    got_keys = f32(keys.download((B, nk, ld)))
+    for b in range(B):
+        for j in range(nk):
+            p = poss[b] - past + j
+            assert np.array_equal(got_keys[b, j, :rank + rd], cached[b, p] if p >= 0 else np.zeros(rank + rd, np.float32))
+    kv_ld = (H * (dim + vdim) + 7) // 8 * 8
+    kv = f32(bf16_bits(rng.standard_normal((B, nk, kv_ld))))
+    q = f32(bf16_bits(rng.standard_normal((B, steps, H, dim + rd))))
+    o_ld = (H * vdim + 7) // 8 * 8
+    dq, dkv, o = dev.from_numpy(bf16_bits(q)), dev.from_numpy(bf16_bits(kv)), dev.zeros(B * steps * o_ld, N.NS_BF16)
+    scale = 1.5 / np.sqrt(dim + rd)
+    N.call("ns_latent_prefill", dev.handle, u(dq.ptr), i64(H * (dim + rd)), u(dkv.ptr), i64(kv_ld), u(keys.ptr), i64(ld), rank, u(st.slots.ptr), u(st.pos.ptr), B, steps,
+           H, dim, rd, vdim, past, window, fl(scale), u(o.ptr), i64(o_ld))
+    dev.synchronize()
+    got = f32(o.download((B, steps, o_ld)))[:, :, :H * vdim].reshape(B, steps, H, vdim)
+    for b in range(B):
+        k = kv[b, :, :H * dim].reshape(nk, H, dim)
+        v = kv[b, :, H * dim:H * (dim + vdim)].reshape(nk, H, vdim)
+        want = np.zeros((steps, H, vdim))
+        for i in range(steps):
+            lo, hi = max(i + past - window + 1, past - poss[b], 0), i + past + 1
+            s = (np.einsum("hd,jhd->hj", q[b, i, :, :dim], k[lo:hi]) + np.einsum("hd,jd->hj", q[b, i, :, dim:], got_keys[b, lo:hi, rank:rank + rd])) * scale
+            s = np.exp(s - s.max(1, keepdims=True))
+            want[i] = np.einsum("hj,jhv->hv", s / s.sum(1, keepdims=True), v[lo:hi])
+        close(got[b], want, 3e-2)
