@@ -184,17 +184,23 @@ class DenseGlu:
 
 
 class DeltaMixer:
-    """Gated delta rule with short convolutions (ns_delta.cu).
+    """Gated delta rule with short convolutions (ns_delta.cu, ns_delta_chunk.cu).
 
     weights: q, k, v, b, o, their convolutions q_conv, k_conv, v_conv, A_log, dt_bias, norm, and either a, g (one decay per head,
     read-out gated by silu) or a1, a2, g1, g2 (one decay per head and key channel through a low-rank pair, read-out gated by the
-    sigmoid of another)."""
+    sigmoid of another).
+
+    A few tokens go through the recurrence one by one, a prompt's portion (bf16 models) in chunks on the tensor cores; the choice
+    depends on the portion's length alone."""
+
+    CHUNK_STEPS = 24         # portions of at least this many tokens are chunked
 
     def __init__(self, ws: Workspace, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float, w: dict):
         assert heads % kv_heads == 0
         self.dev, self.ws, self.eps = ws.dev, ws, eps
         self.heads, self.kv_heads, self.dim, self.vdim, self.taps = heads, kv_heads, dim, vdim, taps
         self.channelwise = "a1" in w
+        self.chunks = ws.dtype == N.NS_BF16 and dim <= 128
         dev = self.dev
         up = lambda a: dev.from_numpy(f32(a).reshape(-1))
         self.conv = [up(w[n + "_conv"]) for n in "qkv"]
@@ -249,7 +255,7 @@ class DeltaMixer:
             a_col, gate_col, act = cols[4], cols[5], N.ACT_SILU
         state: Reservation = cache["state"]
         u = C.c_uint64
-        N.call("ns_delta_recurrent", hd, u(ws["conv_q"]), self.channels[0], u(ws["conv_k"]), self.channels[1], u(ws["conv_v"]), self.channels[2],
+        N.call("ns_delta_chunked" if self.chunks and step.steps >= self.CHUNK_STEPS else "ns_delta_recurrent", hd, u(ws["conv_q"]), self.channels[0], u(ws["conv_k"]), self.channels[1], u(ws["conv_v"]), self.channels[2],
                u(s.ptr), s.splits, s.ld, a_col, u(beta.ptr), beta.splits, beta.ld, beta_col, u(self.a_log.ptr), u(self.dt_bias.ptr), int(self.channelwise),
                u(state.ptr), C.c_int64(state.stride), u(step.slots), step.batch, step.steps, H, self.kv_heads, self.dim, self.vdim, u(ws["read"]), H * self.vdim)
         N.call("ns_gated_norm", hd, u(ws["read"]), H * self.vdim, *s.args, gate_col, act, u(self.norm.ptr), C.c_float(self.eps), C.c_int64(step.m), H, self.vdim,
@@ -289,7 +295,7 @@ class LatentAttentionMixer:
         # its input rows are whole cached rows: the columns of the rotated part are zero
         self.kv = Product(ws, *(np.pad(w[n], ((0, 0), (0, rot_dim))) for n in ("uk", "uv")))
         self.out = Product(ws, w["o"])
-        self.expands = ws.dtype == N.NS_BF16 and vdim <= 256 and dim + rot_dim <= 512
+        self.expands = ws.dtype == N.NS_BF16 and vdim <= 256 and dim + rot_dim <= 256
         ws.need("cq", self.uq.k_ld)
         ws.need("plain", heads * dim)
         ws.need("carried", heads * self.width)

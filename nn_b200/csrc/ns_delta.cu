@@ -43,6 +43,111 @@ struct ConvArgs {
 // The raw inputs of the last taps - 1 tokens are the carried state.  They sit at position modulo taps: a step of one token
 // writes the one place that none of the taps - 1 earlier inputs occupies.  Of a longer step the CTA of the first chunk both
 // reads the history and, after a barrier, replaces it; no other CTA touches these channels' history.
+// V neighbouring channels of a head per lane (32 * V covers the head), up to TAPS taps.  A warp takes CONV_WARP tokens of one head and
+// slides over them with the last inputs in registers, so every input is read once plus taps - 1 at the seam.  `span` warps of a
+// CTA share a head: 4 for prompts, 1 for the few tokens of a decoding step (the CTA then holds four heads).
+constexpr int CONV_WARP = 8;
+
+template <int V>
+NS_DEVINL void conv_load(const NsSource& s, int64_t idx, float (&x)[V])
+{
+    if constexpr (V == 4) {
+        const float4 t = ns_source_at4(s, idx);
+        x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i++) x[i] = ns_source_at(s, idx + i);
+    }
+}
+
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs a, int span, int units)
+{
+    ns_pdl_wait();
+    ns_pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, b = blockIdx.z;
+    int u = span == 4 ? (int)blockIdx.y : (int)blockIdx.y * 4 + warp, s = 0;
+    const bool live = u < units;
+    if (!live) u = 0;
+    while (s + 1 < a.segments && u >= a.seg[s].heads) { u -= a.seg[s].heads; s++; }
+    const ConvSegment& g = a.seg[s];
+    const int slot = a.slots[b], pos0 = a.pos[slot];
+    const int channels = g.heads * g.hd, taps = g.taps, c = lane * V, ch = u * g.hd + c;
+    const bool mine = live && c < g.hd;
+    float* hist = g.hist + (int64_t)slot * a.hist_slot_stride + ch;
+    const int64_t src0 = (int64_t)b * a.steps * a.src.ld + g.col + ch;
+    const int t0 = span == 4 ? ((int)blockIdx.x * 4 + warp) * CONV_WARP : (int)blockIdx.x * CONV_WARP, t1 = min(t0 + CONV_WARP, a.steps);
+    float w[TAPS][V], x[TAPS][V];      // w[n]: weight of the input n tokens back; x[n]: that input
+#pragma unroll
+    for (int n = 0; n < TAPS; n++)
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            w[n][i] = mine && n < taps ? __ldg(g.w + (int64_t)(ch + i) * taps + taps - 1 - n) : 0.0f;
+            x[n][i] = 0.0f;
+        }
+    if (mine && t0 < t1) {
+        // x[n - 1] becomes x[n] before the first token is loaded
+#pragma unroll
+        for (int n = 1; n < TAPS; n++) {
+            const int tt = t0 - n;
+            if (n >= taps || pos0 + tt < 0) continue;
+            if (tt >= 0) {
+                conv_load<V>(a.src, src0 + (int64_t)tt * a.src.ld, x[n - 1]);
+            } else {
+                const float* p = hist + (int64_t)((pos0 + tt) % taps) * channels;
+#pragma unroll
+                for (int i = 0; i < V; i++) x[n - 1][i] = p[i];
+            }
+        }
+    }
+    // all inputs of the warp's tokens are on their way before the first is used
+    float in[CONV_WARP][V];
+#pragma unroll
+    for (int j = 0; j < CONV_WARP; j++)
+        if (mine && t0 + j < t1) conv_load<V>(a.src, src0 + (int64_t)(t0 + j) * a.src.ld, in[j]);
+#pragma unroll
+    for (int j = 0; j < CONV_WARP; j++) {
+        const int t = t0 + j;
+        if (t >= t1) break;
+#pragma unroll
+        for (int n = TAPS - 1; n > 0; n--)
+#pragma unroll
+            for (int i = 0; i < V; i++) x[n][i] = x[n - 1][i];
+#pragma unroll
+        for (int i = 0; i < V; i++) x[0][i] = mine ? in[j][i] : 0.0f;
+        float y[V], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            float acc = 0.0f;
+#pragma unroll
+            for (int n = TAPS - 1; n >= 0; n--) acc = fmaf(x[n][i], w[n][i], acc);
+            y[i] = mine ? ns_silu(acc) : 0.0f;
+            ss = fmaf(y[i], y[i], ss);
+        }
+        float f = 1.0f;
+        if (g.unit) f = g.scale / sqrtf(ns_warp_sum(ss) + 1e-6f);
+        if (mine) {
+            T* out = reinterpret_cast<T*>(g.out) + ((int64_t)b * a.steps + t) * g.out_ld + ch;
+            if constexpr (V == 4) {
+                ns_store4(out, make_float4(y[0] * f, y[1] * f, y[2] * f, y[3] * f));
+            } else {
+#pragma unroll
+                for (int i = 0; i < V; i++) ns_store(out + i, y[i] * f);
+            }
+        }
+    }
+    // the warps that read the history have their inputs: the first `span` warps' tokens come first in the step
+    if (span == 4) __syncthreads();
+    else __syncwarp();
+    if (blockIdx.x != 0 || (span == 4 && warp != 0) || !mine || taps < 2) return;
+    for (int t = max(0, a.steps - (taps - 1)); t < a.steps; t++) {
+        float v[V];
+        conv_load<V>(a.src, src0 + (int64_t)t * a.src.ld, v);
+#pragma unroll
+        for (int i = 0; i < V; i++) hist[(int64_t)((pos0 + t) % taps) * channels + i] = v[i];
+    }
+}
+
 template <typename T, int NV>
 __global__ void __launch_bounds__(128) ns_short_conv_kernel(const ConvArgs a)
 {
@@ -265,29 +370,48 @@ __global__ void __launch_bounds__(256) ns_delta_recurrent_kernel(const DeltaArgs
 // ---------------------------------------------------------------------------------------------
 // y = o / sqrt(mean(o^2) + eps) * w * act(gate), per row and head
 // ---------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) ns_gated_norm_kernel(const float* __restrict__ o, int o_ld, const NsSource gate, int gate_col, int act,
                                                             const float* __restrict__ w, float eps, int64_t rows, int heads, int vdim, T* __restrict__ y,
                                                             int64_t y_ld)
 {
     ns_pdl_wait();
     ns_pdl_trigger();
-    const int64_t item = blockIdx.x * 8ll + (threadIdx.x >> 5);
-    if (item >= rows * heads) return;
-    const int64_t row = item / heads;
-    const int head = (int)(item - row * heads), lane = threadIdx.x & 31;
-    const float* x = o + row * o_ld + (int64_t)head * vdim;
-    float ss = 0.0f;
-    for (int c = lane; c < vdim; c += 32) ss = fmaf(x[c], x[c], ss);
-    const float inv = 1.0f / sqrtf(ns_warp_sum(ss) / (float)vdim + eps);
-    const int64_t gi = row * gate.ld + gate_col + head * vdim;
-    T* out = y + row * y_ld + (int64_t)head * vdim;
-    for (int c = lane; c < vdim; c += 32) {
-        const float z = ns_source_at(gate, gi + c);
-        ns_store(out + c, x[c] * inv * w[c] * (act == NS_ACT_SILU ? ns_silu(z) : ns_sigmoid(z)));
+    const int lane = threadIdx.x & 31;
+    for (int64_t item = blockIdx.x * 8ll + (threadIdx.x >> 5); item < rows * heads; item += gridDim.x * 8ll) {
+        const int64_t row = item / heads;
+        const int head = (int)(item - row * heads);
+        const float* x = o + row * o_ld + (int64_t)head * vdim;
+        const int64_t gi = row * gate.ld + gate_col + head * vdim;
+        T* out = y + row * y_ld + (int64_t)head * vdim;
+        float ss = 0.0f;
+        if (VEC) {
+            // up to 128 values: four per lane
+            const int c = lane * 4;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f), z = v;
+            if (c < vdim) {
+                v = *reinterpret_cast<const float4*>(x + c);
+                z = ns_source_at4(gate, gi + c);
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+            }
+            const float inv = 1.0f / sqrtf(ns_warp_sum(ss) / (float)vdim + eps);
+            if (c < vdim) {
+                const float4 ww = __ldg(reinterpret_cast<const float4*>(w + c));
+                const float4 r = act == NS_ACT_SILU ? make_float4(ns_silu(z.x), ns_silu(z.y), ns_silu(z.z), ns_silu(z.w))
+                                                    : make_float4(ns_sigmoid(z.x), ns_sigmoid(z.y), ns_sigmoid(z.z), ns_sigmoid(z.w));
+                ns_store4(out + c, make_float4(v.x * inv * ww.x * r.x, v.y * inv * ww.y * r.y, v.z * inv * ww.z * r.z, v.w * inv * ww.w * r.w));
+            }
+        } else {
+            for (int c = lane; c < vdim; c += 32) ss = fmaf(x[c], x[c], ss);
+            const float inv = 1.0f / sqrtf(ns_warp_sum(ss) / (float)vdim + eps);
+            for (int c = lane; c < vdim; c += 32) {
+                const float z = ns_source_at(gate, gi + c);
+                ns_store(out + c, x[c] * inv * w[c] * (act == NS_ACT_SILU ? ns_silu(z) : ns_sigmoid(z)));
+            }
+        }
+        if (head == heads - 1)
+            for (int64_t c = (int64_t)heads * vdim + lane; c < y_ld; c += 32) ns_store(y + row * y_ld + c, 0.0f);
     }
-    if (head == heads - 1)
-        for (int64_t c = (int64_t)heads * vdim + lane; c < y_ld; c += 32) ns_store(y + row * y_ld + c, 0.0f);
 }
 
 template <int RPW, int V>
@@ -356,6 +480,32 @@ extern "C" int ns_short_conv(ns_device_t h, uint64_t src, int splits, int src_dt
         NS_CUDA(ns_launch_plain(k, grid, dim3(128), 0, d->stream, a));
         return NS_OK;
     };
+    // the sliding kernel: heads of up to 128 channels, up to 8 taps (its first chunk must hold all tokens that read the history)
+    int most_taps = 1, v = widest <= 32 ? 1 : (widest <= 64 ? 2 : 4);
+    for (int i = 0; i < segments; i++) {
+        const ConvSegment& s = a.seg[i];
+        if (s.taps > most_taps) most_taps = s.taps;
+        if (s.hd % v != 0 || (v == 4 && ((s.col | s.out_ld) & 3) != 0)) v = 0;
+        if (v == 4 && (reinterpret_cast<uintptr_t>(s.out) & 15) != 0) v = 0;
+        if (v == 0) break;
+    }
+    if (v == 4 && ((src_ld & 3) != 0 || (src & 15) != 0)) v = 0;
+    if (v != 0 && widest <= 128 && most_taps <= 8) {
+        const int span = steps <= CONV_WARP ? 1 : 4;
+        const int per = span * CONV_WARP;
+        const dim3 sgrid((unsigned)((steps + per - 1) / per), (unsigned)(span == 4 ? units : (units + 3) / 4), (unsigned)batch);
+        auto slide = [&](auto k) -> int {
+            NS_CUDA(ns_launch_plain(k, sgrid, dim3(128), 0, d->stream, a, span, units));
+            return NS_OK;
+        };
+        auto pick = [&](auto zero) -> int {
+            using T = decltype(zero);
+            if (most_taps <= 4)
+                return v == 1 ? slide(ns_short_conv_slide_kernel<T, 1, 4>) : (v == 2 ? slide(ns_short_conv_slide_kernel<T, 2, 4>) : slide(ns_short_conv_slide_kernel<T, 4, 4>));
+            return v == 1 ? slide(ns_short_conv_slide_kernel<T, 1, 8>) : (v == 2 ? slide(ns_short_conv_slide_kernel<T, 2, 8>) : slide(ns_short_conv_slide_kernel<T, 4, 8>));
+        };
+        return out_dtype == NS_F32 ? pick(float(0)) : pick(uint16_t(0));
+    }
     if (out_dtype == NS_F32) {
         if (widest <= 64) return launch(ns_short_conv_kernel<float, 2>);
         if (widest <= 128) return launch(ns_short_conv_kernel<float, 4>);
@@ -405,12 +555,17 @@ extern "C" int ns_gated_norm(ns_device_t h, uint64_t o, int o_ld, uint64_t gate,
     NS_REQUIRE(act == NS_ACT_SILU || act == NS_ACT_SIGMOID, NS_ERR_ARGUMENT, "ns_gated_norm: unknown activation %d", act);
     NS_REQUIRE(out_dtype == NS_F32 || out_dtype == NS_BF16, NS_ERR_ARGUMENT, "ns_gated_norm: bad output type");
     const NsSource g = ns_source(gate, splits, gate_dtype, rows, gate_ld);
-    const unsigned grid = (unsigned)((rows * heads + 7) / 8);
-    if (out_dtype == NS_F32)
-        NS_CUDA(ns_launch_plain(ns_gated_norm_kernel<float>, dim3(grid), dim3(256), 0, d->stream, reinterpret_cast<const float*>(o), o_ld, g, gate_col, act,
-                                reinterpret_cast<const float*>(w), eps, rows, heads, vdim, reinterpret_cast<float*>(y), (int64_t)y_ld));
-    else
-        NS_CUDA(ns_launch_plain(ns_gated_norm_kernel<uint16_t>, dim3(grid), dim3(256), 0, d->stream, reinterpret_cast<const float*>(o), o_ld, g, gate_col, act,
-                                reinterpret_cast<const float*>(w), eps, rows, heads, vdim, reinterpret_cast<uint16_t*>(y), (int64_t)y_ld));
+    const bool vec = vdim <= 128 && ((vdim | o_ld | gate_ld | gate_col | y_ld) & 3) == 0 && ((o | gate | w | y) & 15) == 0;
+    const int64_t blocks = (rows * heads + 7) / 8, most = (int64_t)d->sm_count * 32;
+    const dim3 grid((unsigned)(blocks < most ? blocks : most));
+    if (out_dtype == NS_F32) {
+        auto k = vec ? ns_gated_norm_kernel<float, true> : ns_gated_norm_kernel<float, false>;
+        NS_CUDA(ns_launch_plain(k, grid, dim3(256), 0, d->stream, reinterpret_cast<const float*>(o), o_ld, g, gate_col, act, reinterpret_cast<const float*>(w), eps,
+                                rows, heads, vdim, reinterpret_cast<float*>(y), (int64_t)y_ld));
+    } else {
+        auto k = vec ? ns_gated_norm_kernel<uint16_t, true> : ns_gated_norm_kernel<uint16_t, false>;
+        NS_CUDA(ns_launch_plain(k, grid, dim3(256), 0, d->stream, reinterpret_cast<const float*>(o), o_ld, g, gate_col, act, reinterpret_cast<const float*>(w), eps,
+                                rows, heads, vdim, reinterpret_cast<uint16_t*>(y), (int64_t)y_ld));
+    }
     return NS_OK;
 }

@@ -35,37 +35,64 @@ struct LatentAppendArgs {
     int ring_len, ring_ld;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(128) ns_latent_append_kernel(const LatentAppendArgs a)
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) ns_latent_append_kernel(const LatentAppendArgs a)
 {
-    __shared__ float red[2][4];
+    extern __shared__ float4 app_smem[];
+    float* x = reinterpret_cast<float*>(app_smem);             // the row
+    __shared__ float red[2][8];
     ns_pdl_wait();
     ns_pdl_trigger();
     const int row = blockIdx.x, b = row / a.steps, i = row % a.steps, tid = threadIdx.x;
     const int slot = a.slots[b], p = a.pos[slot] + i;
     const int64_t base = (int64_t)row * a.src.ld;
+    const int k1 = a.q_rank + a.kv_rank, n = k1 + a.rot_dim;
     float sq = 0.0f, sc = 0.0f;
-    for (int c = tid; c < a.q_rank; c += 128) { const float v = ns_source_at(a.src, base + c); sq = fmaf(v, v, sq); }
-    for (int c = tid; c < a.kv_rank; c += 128) { const float v = ns_source_at(a.src, base + a.q_rank + c); sc = fmaf(v, v, sc); }
+    auto sum = [&](int c, float v) {
+        if (c < a.q_rank) sq = fmaf(v, v, sq);
+        else if (c < k1) sc = fmaf(v, v, sc);
+    };
+    if (VEC) {
+        for (int c = tid * 4; c < n; c += 1024) {
+            const float4 v = ns_source_at4(a.src, base + c);
+            *reinterpret_cast<float4*>(x + c) = v;
+            sum(c, v.x); sum(c + 1, v.y); sum(c + 2, v.z); sum(c + 3, v.w);
+        }
+    } else {
+        for (int c = tid; c < n; c += 256) {
+            x[c] = ns_source_at(a.src, base + c);
+            sum(c, x[c]);
+        }
+    }
     const float iq = 1.0f / sqrtf(ns_cta_sum(sq, red[0]) / (float)a.q_rank + a.eps);
     const float ic = 1.0f / sqrtf(ns_cta_sum(sc, red[1]) / (float)a.kv_rank + a.eps);
     T* cq = reinterpret_cast<T*>(a.cq) + (int64_t)row * a.cq_ld;
-    for (int c = tid; c < a.cq_ld; c += 128) ns_store(cq + c, c < a.q_rank ? ns_source_at(a.src, base + c) * iq * a.q_norm[c] : 0.0f);
     T* dst = reinterpret_cast<T*>(a.ring) + (int64_t)slot * a.ring_slot_stride + (int64_t)(p % a.ring_len) * a.ring_ld;
-    for (int c = tid; c < a.kv_rank; c += 128) ns_store(dst + c, ns_source_at(a.src, base + a.q_rank + c) * ic * a.kv_norm[c]);
-    const int64_t rb = base + a.q_rank + a.kv_rank;
-    for (int c = tid; c < a.rot_dim; c += 128) {
-        const float x = ns_source_at(a.src, rb + c);
-        float y = x;
-        if (c < a.rot_dims) {
-            float sn, cs;
-            sincosf((float)p * a.freq[c >> 1], &sn, &cs);
-            const float other = ns_source_at(a.src, rb + (c ^ 1));
-            y = (c & 1) ? fmaf(x, cs, other * sn) : fmaf(x, cs, -other * sn);
+    const float* xc = x + a.q_rank;
+    if (VEC) {
+        for (int c = tid * 4; c < a.q_rank; c += 1024) {
+            const float4 w = __ldg(reinterpret_cast<const float4*>(a.q_norm + c));
+            ns_store4(cq + c, make_float4(x[c] * iq * w.x, x[c + 1] * iq * w.y, x[c + 2] * iq * w.z, x[c + 3] * iq * w.w));
         }
-        ns_store(dst + a.kv_rank + c, y);
+        for (int c = tid * 4; c < a.kv_rank; c += 1024) {
+            const float4 w = __ldg(reinterpret_cast<const float4*>(a.kv_norm + c));
+            ns_store4(dst + c, make_float4(xc[c] * ic * w.x, xc[c + 1] * ic * w.y, xc[c + 2] * ic * w.z, xc[c + 3] * ic * w.w));
+        }
+    } else {
+        for (int c = tid; c < a.q_rank; c += 256) ns_store(cq + c, x[c] * iq * a.q_norm[c]);
+        for (int c = tid; c < a.kv_rank; c += 256) ns_store(dst + c, xc[c] * ic * a.kv_norm[c]);
     }
-    for (int c = a.kv_rank + a.rot_dim + tid; c < a.ring_ld; c += 128) ns_store(dst + c, 0.0f);
+    for (int c = a.q_rank + tid; c < a.cq_ld; c += 256) ns_store(cq + c, 0.0f);
+    // a thread per pair, then what passes unturned
+    const float* xr = x + k1;
+    for (int c = 2 * (255 - tid); c < a.rot_dims; c += 512) {
+        float sn, cs;
+        sincosf((float)p * a.freq[c >> 1], &sn, &cs);
+        ns_store(dst + a.kv_rank + c, fmaf(xr[c], cs, -xr[c + 1] * sn));
+        ns_store(dst + a.kv_rank + c + 1, fmaf(xr[c + 1], cs, xr[c] * sn));
+    }
+    for (int c = a.rot_dims + tid; c < a.rot_dim; c += 256) ns_store(dst + a.kv_rank + c, xr[c]);
+    for (int c = a.kv_rank + a.rot_dim + tid; c < a.ring_ld; c += 256) ns_store(dst + c, 0.0f);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -82,7 +109,7 @@ struct RotateArgs {
     void* rot; int64_t rot_ld; int rot_head;
 };
 
-template <typename TP, typename TR>
+template <typename TP, typename TR, bool VEC>
 __global__ void __launch_bounds__(256) ns_rotate_heads_kernel(const RotateArgs a)
 {
     extern __shared__ float2 cs[];
@@ -97,6 +124,26 @@ __global__ void __launch_bounds__(256) ns_rotate_heads_kernel(const RotateArgs a
     }
     __syncthreads();
     const int w = a.dim + a.rot_dim, n = a.heads * w;
+    if (VEC) {
+        for (int e = threadIdx.x * 4; e < n; e += blockDim.x * 4) {
+            const int head = e / w, c = e - head * w, r = c - a.dim;
+            float4 v = ns_source_at4(a.src, (int64_t)row * a.src.ld + e);
+            if (r < 0) {
+                ns_store4(reinterpret_cast<TP*>(a.plain) + (int64_t)row * a.plain_ld + (int64_t)head * a.plain_head + c, v);
+                continue;
+            }
+            if (r < a.rot_dims) {
+                const float2 s = cs[r >> 1];
+                v = make_float4(fmaf(v.x, s.x, -v.y * s.y), fmaf(v.y, s.x, v.x * s.y), v.z, v.w);
+            }
+            if (r + 2 < a.rot_dims) {
+                const float2 t = cs[(r >> 1) + 1];
+                v = make_float4(v.x, v.y, fmaf(v.z, t.x, -v.w * t.y), fmaf(v.w, t.x, v.z * t.y));
+            }
+            ns_store4(reinterpret_cast<TR*>(a.rot) + (int64_t)row * a.rot_ld + (int64_t)head * a.rot_head + r, v);
+        }
+        return;
+    }
     for (int e = threadIdx.x; e < n; e += blockDim.x) {
         const int head = e / w, c = e - head * w;
         const int64_t at = (int64_t)row * a.src.ld + e;
@@ -304,8 +351,12 @@ extern "C" int ns_latent_append(ns_device_t h, uint64_t src, int splits, int src
     a.slots = I32P(slots); a.pos = I32P(pos); a.steps = steps;
     a.cq = reinterpret_cast<void*>(cq); a.cq_ld = cq_ld;
     a.ring = reinterpret_cast<void*>(ring); a.ring_slot_stride = ring_slot_stride; a.ring_len = ring_len; a.ring_ld = ring_ld;
-    auto k = dtype == NS_F32 ? ns_latent_append_kernel<float> : ns_latent_append_kernel<uint16_t>;
-    NS_CUDA(ns_launch_plain(k, dim3((unsigned)(batch * steps)), dim3(128), 0, d->stream, a));
+    const int n = q_rank + kv_rank + rot_dim;
+    NS_REQUIRE(n <= 12000, NS_ERR_ARGUMENT, "ns_latent_append: rows of %d values do not fit shared memory", n);
+    const bool vec = ((q_rank | kv_rank | rot_dim | src_ld | cq_ld | ring_ld) & 3) == 0 && (ring_slot_stride & 3) == 0 && ((src | q_norm | kv_norm | cq | ring) & 15) == 0;
+    auto k = dtype == NS_F32 ? (vec ? ns_latent_append_kernel<float, true> : ns_latent_append_kernel<float, false>)
+                             : (vec ? ns_latent_append_kernel<uint16_t, true> : ns_latent_append_kernel<uint16_t, false>);
+    NS_CUDA(ns_launch_plain(k, dim3((unsigned)(batch * steps)), dim3(256), (size_t)((n + 3) & ~3) * 4, d->stream, a));
     return NS_OK;
 }
 
@@ -325,10 +376,16 @@ extern "C" int ns_rotate_heads(ns_device_t h, uint64_t src, int splits, int src_
     a.slots = I32P(slots); a.pos = I32P(pos); a.steps = steps;
     a.plain = reinterpret_cast<void*>(plain); a.plain_ld = plain_ld; a.plain_head = plain_head;
     a.rot = reinterpret_cast<void*>(rot); a.rot_ld = rot_ld; a.rot_head = rot_head;
-    auto k = plain_dtype == NS_F32 ? (rot_dtype == NS_F32 ? ns_rotate_heads_kernel<float, float> : ns_rotate_heads_kernel<float, uint16_t>)
-                                   : (rot_dtype == NS_F32 ? ns_rotate_heads_kernel<uint16_t, float> : ns_rotate_heads_kernel<uint16_t, uint16_t>);
-    NS_CUDA(ns_launch_plain(k, dim3((unsigned)(batch * steps)), dim3(256), (size_t)(rot_dims / 2 + 1) * sizeof(float2), d->stream, a));
-    return NS_OK;
+    const bool vec = ((dim | rot_dim | src_ld | plain_head | rot_head) & 3) == 0 && ((plain_ld | rot_ld) & 3) == 0 &&
+                     (src & 15) == 0 && (plain & (plain_dtype == NS_F32 ? 15 : 7)) == 0 && (rot & (rot_dtype == NS_F32 ? 15 : 7)) == 0;
+    auto go = [&](auto kern) -> int {
+        NS_CUDA(ns_launch_plain(kern, dim3((unsigned)(batch * steps)), dim3(256), (size_t)(rot_dims / 2 + 1) * sizeof(float2), d->stream, a));
+        return NS_OK;
+    };
+    if (plain_dtype == NS_F32 && rot_dtype == NS_F32) return vec ? go(ns_rotate_heads_kernel<float, float, true>) : go(ns_rotate_heads_kernel<float, float, false>);
+    if (plain_dtype == NS_BF16 && rot_dtype == NS_BF16)
+        return vec ? go(ns_rotate_heads_kernel<uint16_t, uint16_t, true>) : go(ns_rotate_heads_kernel<uint16_t, uint16_t, false>);
+    return ns_fail(NS_ERR_ARGUMENT, "ns_rotate_heads: both outputs have one type");
 }
 
 extern "C" int ns_head_matmul(ns_device_t h, int x_dtype, uint64_t x, int64_t x_ld, int x_head, int w_dtype, uint64_t w, int64_t w_head, int64_t w_k, int64_t w_n,

@@ -47,18 +47,20 @@ struct PrefillArgs {
     const int32_t* pos;
     int steps, heads, dim, rot, vdim, past, nk, window;
     float scale2;                            // scale * log2(e)
-    int dkp, vec;
+    int vec;
 };
 
 constexpr int PF_ROWS = 64, PF_KEYS = 64;
 
-template <int NV>      // value n-tiles of 8
+// NV: value n-tiles of 8.  KS: 16-wide k-steps of the scores whose query fragments stay in registers.
+template <int NV, int KS>
 __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArgs a)
 {
     extern __shared__ __align__(16) uint16_t pf_smem[];
-    constexpr int VLD = NV * 8 + 8;
-    const int kld = a.dkp + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-    const uint32_t sQ = ns_smem_u32(pf_smem), sK = sQ + PF_ROWS * kld * 2, sV = sK + 2 * PF_KEYS * kld * 2;
+    constexpr int VLD = NV * 8 + 8, DKP = KS * 16, KLD = DKP + 8;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const uint32_t sK = ns_smem_u32(pf_smem), sV = sK + 2 * PF_KEYS * KLD * 2;
+    const uint32_t sQ = sK + PF_KEYS * KLD * 2;          // the second key stage, before it is filled
     ns_pdl_wait();
     ns_pdl_trigger();
     const int tiles_q = (a.steps + PF_ROWS - 1) / PF_ROWS;
@@ -66,42 +68,46 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
     const int pos0 = a.pos[a.slots[b]];
     const int dk = a.dim + a.rot;
 
-    for (int e = tid; e < PF_ROWS * (a.dkp / 8); e += 128) {
-        const int r = e / (a.dkp / 8), c = (e - r * (a.dkp / 8)) * 8;
+    // a warp per row, a lane per 16 bytes
+    for (int r = warp; r < PF_ROWS; r += 4) {
         const bool in = q0 + r < a.steps;
-        ns_copy8(sQ + (r * kld + c) * 2, a.q + ((int64_t)b * a.steps + (in ? q0 + r : 0)) * a.q_ld + (int64_t)head * dk + c, in ? dk - c : 0, a.vec);
+        const uint16_t* src = a.q + ((int64_t)b * a.steps + (in ? q0 + r : 0)) * a.q_ld + (int64_t)head * dk;
+        for (int c = lane * 8; c < DKP; c += 256) ns_copy8(sQ + (r * KLD + c) * 2, src + (in && c < dk ? c : 0), in ? dk - c : 0, a.vec);
     }
     auto load_tile = [&](int kt, int stage) {
         const int k0 = kt * PF_KEYS;
-        const uint32_t dk_s = sK + stage * PF_KEYS * kld * 2, dv_s = sV + stage * PF_KEYS * VLD * 2;
-        for (int e = tid; e < PF_KEYS * (a.dkp / 8); e += 128) {
-            const int r = e / (a.dkp / 8), c = (e - r * (a.dkp / 8)) * 8;
-            const int64_t row = (int64_t)b * a.nk + k0 + r;
+        const uint32_t dk_s = sK + stage * PF_KEYS * KLD * 2, dv_s = sV + stage * PF_KEYS * VLD * 2;
+        for (int r = warp; r < PF_KEYS; r += 4) {
             const bool in = k0 + r < a.nk;
-            const uint32_t dst = dk_s + (r * kld + c) * 2;
-            if (a.vec) {
-                if (c < a.dim) ns_copy8(dst, a.kv + (in ? row : 0) * a.kv_ld + (int64_t)head * a.dim + c, in ? 8 : 0, true);
-                else ns_copy8(dst, a.keys + (in ? row : 0) * a.keys_ld + a.rank + c - a.dim, in ? dk - c : 0, true);
-            } else {
-                uint32_t w[4];
+            const int64_t row = (int64_t)b * a.nk + (in ? k0 + r : 0);
+            const uint16_t* kp = a.kv + row * a.kv_ld + (int64_t)head * a.dim;
+            const uint16_t* rp = a.keys + row * a.keys_ld + a.rank;
+            for (int c = lane * 8; c < DKP; c += 256) {
+                const uint32_t dst = dk_s + (r * KLD + c) * 2;
+                if (a.vec) {
+                    const uint16_t* src = c < a.dim ? kp + c : rp + (c < dk ? c - a.dim : 0);
+                    ns_copy8(dst, src, in ? dk - c : 0, true);
+                } else {
+                    uint32_t w[4];
 #pragma unroll
-                for (int i = 0; i < 4; i++) {
-                    uint32_t h2[2];
+                    for (int i = 0; i < 4; i++) {
+                        uint32_t h2[2];
 #pragma unroll
-                    for (int s = 0; s < 2; s++) {
-                        const int cc = c + 2 * i + s;
-                        h2[s] = !in || cc >= dk ? 0u : (cc < a.dim ? a.kv[row * a.kv_ld + (int64_t)head * a.dim + cc] : a.keys[row * a.keys_ld + a.rank + cc - a.dim]);
+                        for (int s = 0; s < 2; s++) {
+                            const int cc = c + 2 * i + s;
+                            h2[s] = !in || cc >= dk ? 0u : (cc < a.dim ? kp[cc] : rp[cc - a.dim]);
+                        }
+                        w[i] = h2[0] | (h2[1] << 16);
                     }
-                    w[i] = h2[0] | (h2[1] << 16);
+                    ns_st_shared_v4(dst, w[0], w[1], w[2], w[3]);
                 }
-                ns_st_shared_v4(dst, w[0], w[1], w[2], w[3]);
             }
         }
         for (int e = tid; e < PF_KEYS * NV; e += 128) {
             const int r = e / NV, c = (e - r * NV) * 8;
-            const int64_t row = (int64_t)b * a.nk + k0 + r;
             const bool in = k0 + r < a.nk;
-            ns_copy8(dv_s + (r * VLD + c) * 2, a.kv + (in ? row : 0) * a.kv_ld + (int64_t)a.heads * a.dim + (int64_t)head * a.vdim + (c < a.vdim ? c : 0),
+            const int64_t row = (int64_t)b * a.nk + (in ? k0 + r : 0);
+            ns_copy8(dv_s + (r * VLD + c) * 2, a.kv + row * a.kv_ld + (int64_t)a.heads * a.dim + (int64_t)head * a.vdim + (c < a.vdim ? c : 0),
                      in ? a.vdim - c : 0, a.vec);
         }
         ns_cp_commit();
@@ -122,6 +128,12 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
     const int r0 = q0 + warp * 16 + g;       // query rows r0 and r0 + 8
 
     load_tile(t_first, 0);
+    ns_cp_wait<0>();
+    __syncthreads();
+    uint32_t qf[KS][4];
+#pragma unroll
+    for (int k = 0; k < KS; k++) ns_ldsm4(qf[k], ns_addr_a(sQ, KLD, warp * 16, k * 16, lane));
+    __syncthreads();
     for (int kt = t_first; kt <= t_last; kt++) {
         const int stage = (kt - t_first) & 1;
         if (kt < t_last) {
@@ -131,21 +143,25 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
             ns_cp_wait<0>();
         }
         __syncthreads();
-        const uint32_t tK = sK + stage * PF_KEYS * kld * 2, tV = sV + stage * PF_KEYS * VLD * 2;
+        const uint32_t tK = sK + stage * PF_KEYS * KLD * 2, tV = sV + stage * PF_KEYS * VLD * 2;
         float s[8][4];
 #pragma unroll
         for (int j = 0; j < 8; j++)
 #pragma unroll
             for (int i = 0; i < 4; i++) s[j][i] = 0.0f;
-        for (int k = 0; k < a.dkp; k += 16) {
-            uint32_t af[4];
-            ns_ldsm4(af, ns_addr_a(sQ, kld, warp * 16, k, lane));
+        // the next k-step's key fragments are on their way while this one is multiplied
+        uint32_t bf[2][4][4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) ns_ldsm4(bf[0][j], ns_addr_b(tK, KLD, j * 16, 0, lane));
+#pragma unroll
+        for (int k = 0; k < KS; k++) {
+            if (k + 1 < KS)
+#pragma unroll
+                for (int j = 0; j < 4; j++) ns_ldsm4(bf[(k + 1) & 1][j], ns_addr_b(tK, KLD, j * 16, (k + 1) * 16, lane));
 #pragma unroll
             for (int j = 0; j < 4; j++) {
-                uint32_t bf[4];
-                ns_ldsm4(bf, ns_addr_b(tK, kld, j * 16, k, lane));
-                ns_mma_bf16(s[2 * j], af, bf[0], bf[1]);
-                ns_mma_bf16(s[2 * j + 1], af, bf[2], bf[3]);
+                ns_mma_bf16(s[2 * j], qf[k], bf[k & 1][j][0], bf[k & 1][j][1]);
+                ns_mma_bf16(s[2 * j + 1], qf[k], bf[k & 1][j][2], bf[k & 1][j][3]);
             }
         }
         const int k0 = kt * PF_KEYS;
@@ -189,16 +205,25 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
         for (int j = 0; j < NV; j++) {
             acc[j][0] *= f[0]; acc[j][1] *= f[0]; acc[j][2] *= f[1]; acc[j][3] *= f[1];
         }
+        constexpr int GV = NV >= 8 ? 4 : NV / 2, NG = NV / 2 / GV;      // value fragments in groups of GV, one group ahead
+        uint32_t vf[2][GV][4];
+#pragma unroll
+        for (int j = 0; j < GV; j++) ns_ldsm4_t(vf[0][j], ns_addr_bt(tV, VLD, 0, j * 16, lane));
 #pragma unroll
         for (int k = 0; k < 4; k++) {
-            uint32_t pf[4] = {ns_pack_bf16x2(s[2 * k][0], s[2 * k][1]), ns_pack_bf16x2(s[2 * k][2], s[2 * k][3]),
-                              ns_pack_bf16x2(s[2 * k + 1][0], s[2 * k + 1][1]), ns_pack_bf16x2(s[2 * k + 1][2], s[2 * k + 1][3])};
+            const uint32_t pf[4] = {ns_pack_bf16x2(s[2 * k][0], s[2 * k][1]), ns_pack_bf16x2(s[2 * k][2], s[2 * k][3]),
+                                    ns_pack_bf16x2(s[2 * k + 1][0], s[2 * k + 1][1]), ns_pack_bf16x2(s[2 * k + 1][2], s[2 * k + 1][3])};
 #pragma unroll
-            for (int j = 0; j < NV / 2; j++) {
-                uint32_t bf[4];
-                ns_ldsm4_t(bf, ns_addr_bt(tV, VLD, k * 16, j * 16, lane));
-                ns_mma_bf16(acc[2 * j], pf, bf[0], bf[1]);
-                ns_mma_bf16(acc[2 * j + 1], pf, bf[2], bf[3]);
+            for (int q = 0; q < NG; q++) {
+                const int at = k * NG + q, nx = at + 1;
+                if (nx < 4 * NG)
+#pragma unroll
+                    for (int j = 0; j < GV; j++) ns_ldsm4_t(vf[nx & 1][j], ns_addr_bt(tV, VLD, (nx / NG) * 16, ((nx % NG) * GV + j) * 16, lane));
+#pragma unroll
+                for (int j = 0; j < GV; j++) {
+                    ns_mma_bf16(acc[2 * (q * GV + j)], pf, vf[at & 1][j][0], vf[at & 1][j][1]);
+                    ns_mma_bf16(acc[2 * (q * GV + j) + 1], pf, vf[at & 1][j][2], vf[at & 1][j][3]);
+                }
             }
         }
         __syncthreads();
@@ -266,19 +291,20 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
     const int tiles = (last - first) / DC_KEYS + 1, per = (tiles + a.splits - 1) / a.splits;
     const int tb = split * per, te = min(tiles, tb + per);
 
-    const int cpr = a.wp / 8;
-    for (int e = tid; e < R * cpr; e += 256) {
-        const int r = e / cpr, c = (e - r * cpr) * 8;
+    for (int r = warp; r < R; r += 8) {
         const bool in = row0 + r < a.rows;
-        ns_copy8(sQ + (r * ld + c) * 2, a.q + ((int64_t)b * a.rows + (in ? row0 + r : 0)) * a.width + c, in ? a.width - c : 0, (a.width & 7) == 0);
+        const uint16_t* src = a.q + ((int64_t)b * a.rows + (in ? row0 + r : 0)) * a.width;
+        for (int c = lane * 8; c < a.wp; c += 256) ns_copy8(sQ + (r * ld + c) * 2, src + (c < a.width ? c : 0), in ? a.width - c : 0, (a.width & 7) == 0);
     }
+    // a warp per cached row; rows are padded to a multiple of 8 with zeros
     auto load_tile = [&](int t, int stage) {
         const int p0 = first + t * DC_KEYS;
-        for (int e = tid; e < DC_KEYS * cpr; e += 256) {
-            const int r = e / cpr, c = (e - r * cpr) * 8;
+#pragma unroll 2
+        for (int r = warp; r < DC_KEYS; r += 8) {
             const bool in = p0 + r <= last;
-            // cached rows are padded to a multiple of 8 with zeros
-            ns_copy8(sC + ((stage * DC_KEYS + r) * ld + c) * 2, ring + (int64_t)(in ? (p0 + r) % a.ring_len : 0) * a.ring_ld + c, in ? a.ring_ld - c : 0, true);
+            const uint16_t* src = ring + (int64_t)(in ? (p0 + r) % a.ring_len : 0) * a.ring_ld;
+            for (int c = lane * 8; c < a.wp; c += 256)
+                ns_copy8(sC + ((stage * DC_KEYS + r) * ld + c) * 2, src + (c < a.ring_ld ? c : 0), in ? a.ring_ld - c : 0, true);
         }
         ns_cp_commit();
     };
@@ -307,23 +333,29 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
         __syncthreads();
         const uint32_t tC = sC + stage * DC_KEYS * ld * 2;
         // scores: warp w takes keys 8w .. 8w + 7
-        float s[MT][4];
+        // two chains of accumulation per row tile
+        float s[MT][4], s2[MT][4];
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
-            for (int k = 0; k < 4; k++) s[i][k] = 0.0f;
+            for (int k = 0; k < 4; k++) s[i][k] = s2[i][k] = 0.0f;
+#pragma unroll 4
         for (int k = 0; k < a.wp; k += 32) {
             uint32_t bf[4];
             ns_ldsm4(bf, tC + ((warp * 8 + (lane & 7)) * ld + k + (lane >> 3) * 8) * 2);
 #pragma unroll
             for (int i = 0; i < MT; i++) {
-                uint32_t af[4];
+                uint32_t af[4], ag[4];
                 ns_ldsm4(af, ns_addr_a(sQ, ld, i * 16, k, lane));
+                ns_ldsm4(ag, ns_addr_a(sQ, ld, i * 16, k + 16, lane));
                 ns_mma_bf16(s[i], af, bf[0], bf[1]);
-                ns_ldsm4(af, ns_addr_a(sQ, ld, i * 16, k + 16, lane));
-                ns_mma_bf16(s[i], af, bf[2], bf[3]);
+                ns_mma_bf16(s2[i], ag, bf[2], bf[3]);
             }
         }
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int k = 0; k < 4; k++) s[i][k] += s2[i][k];
         const int p0 = first + t * DC_KEYS;
 #pragma unroll
         for (int i = 0; i < MT; i++)
@@ -503,15 +535,25 @@ __global__ void __launch_bounds__(128) ns_head_matmul_tc_kernel(const HeadTcArgs
         }
 }
 
-template <int NV>
+template <int NV, int KS>
 int launch_prefill(NsDevice* d, const PrefillArgs& a, int batch)
 {
-    const size_t smem = ((size_t)(PF_ROWS + 2 * PF_KEYS) * (a.dkp + 8) + 2 * PF_KEYS * (NV * 8 + 8)) * 2;
-    NS_REQUIRE(smem <= 227 * 1024, NS_ERR_ARGUMENT, "ns_latent_prefill: heads of %d + %d do not fit shared memory", a.dkp, a.vdim);
-    auto k = ns_latent_prefill_kernel<NV>;
+    constexpr size_t smem = ((size_t)2 * PF_KEYS * (KS * 16 + 8) + 2 * PF_KEYS * (NV * 8 + 8)) * 2;
+    static_assert(smem <= 227 * 1024, "tiles do not fit shared memory");
+    auto k = ns_latent_prefill_kernel<NV, KS>;
     NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     NS_CUDA(ns_launch_plain(k, dim3((a.steps + PF_ROWS - 1) / PF_ROWS, a.heads, batch), dim3(128), smem, d->stream, a));
     return NS_OK;
+}
+
+template <int NV>
+int dispatch_prefill(NsDevice* d, const PrefillArgs& a, int batch)
+{
+    const int dk = a.dim + a.rot;
+    if (dk <= 64) return launch_prefill<NV, 4>(d, a, batch);
+    if (dk <= 128) return launch_prefill<NV, 8>(d, a, batch);
+    if (dk <= 192) return launch_prefill<NV, 12>(d, a, batch);
+    return launch_prefill<NV, 16>(d, a, batch);
 }
 
 template <int MT, int NW>
@@ -556,7 +598,7 @@ extern "C" int ns_latent_prefill(ns_device_t h, uint64_t q, int64_t q_ld, uint64
     NS_ENTER(h);
     NS_REQUIRE(q && kv && keys && slots && pos && o && batch > 0 && batch <= 65535 && steps > 0 && heads > 0 && heads <= 65535, NS_ERR_ARGUMENT,
                "ns_latent_prefill: bad argument");
-    NS_REQUIRE(dim > 0 && rot_dim >= 0 && vdim > 0 && vdim <= 256 && rank > 0 && past >= 0 && window >= 0, NS_ERR_ARGUMENT, "ns_latent_prefill: bad sizes");
+    NS_REQUIRE(dim > 0 && rot_dim >= 0 && dim + rot_dim <= 256 && vdim > 0 && vdim <= 256 && rank > 0 && past >= 0 && window >= 0, NS_ERR_ARGUMENT, "ns_latent_prefill: bad sizes");
     NS_REQUIRE(kv_ld >= (int64_t)heads * (dim + vdim) && q_ld >= (int64_t)heads * (dim + rot_dim) && keys_ld >= rank + rot_dim && o_ld >= (int64_t)heads * vdim,
                NS_ERR_ARGUMENT, "ns_latent_prefill: rows too short");
     PrefillArgs a;
@@ -564,12 +606,11 @@ extern "C" int ns_latent_prefill(ns_device_t h, uint64_t q, int64_t q_ld, uint64
     a.o = reinterpret_cast<uint16_t*>(o); a.o_ld = o_ld; a.slots = I32P(slots); a.pos = I32P(pos);
     a.steps = steps; a.heads = heads; a.dim = dim; a.rot = rot_dim; a.vdim = vdim; a.past = past; a.nk = past + steps; a.window = window;
     a.scale2 = scale * LOG2E;
-    a.dkp = (dim + rot_dim + 15) / 16 * 16;
     a.vec = ((dim | rot_dim | vdim | rank | (int)q_ld | (int)kv_ld | (int)keys_ld) & 7) == 0 && ((q | kv | keys) & 15) == 0;
-    if (vdim <= 32) return launch_prefill<4>(d, a, batch);
-    if (vdim <= 64) return launch_prefill<8>(d, a, batch);
-    if (vdim <= 128) return launch_prefill<16>(d, a, batch);
-    return launch_prefill<32>(d, a, batch);
+    if (vdim <= 32) return dispatch_prefill<4>(d, a, batch);
+    if (vdim <= 64) return dispatch_prefill<8>(d, a, batch);
+    if (vdim <= 128) return dispatch_prefill<16>(d, a, batch);
+    return dispatch_prefill<32>(d, a, batch);
 }
 
 extern "C" int ns_latent_decode(ns_device_t h, uint64_t q, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld, int rank, int width, int window,
@@ -593,7 +634,7 @@ extern "C" int ns_latent_decode(ns_device_t h, uint64_t q, uint64_t ring, int64_
     NS_REQUIRE((a.rows + R - 1) / R <= 65535, NS_ERR_ARGUMENT, "ns_latent_decode: too many rows");
     // about one CTA per SM (the two tiles in flight fill its shared memory), at least two tiles of keys each
     const int span = window > 0 ? window - 1 + steps : ring_len;
-    int splits = (int)((d->sm_count + ctas - 1) / ctas);
+    int splits = (int)(d->sm_count / ctas);
     const int most = (span / DC_KEYS + 1) / 2;
     if (splits > most) splits = most;
     if (splits > 16) splits = 16;

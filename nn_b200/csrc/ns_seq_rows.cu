@@ -12,7 +12,14 @@ namespace {
 // ---------------------------------------------------------------------------------------------
 // y[b, i, :] = scale * table[token] + bigram[row(previous token, token)]
 // ---------------------------------------------------------------------------------------------
-template <typename T>
+NS_DEVINL float4 embed_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+NS_DEVINL float4 embed_load4(const uint16_t* p)
+{
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xFFFF0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xFFFF0000u));
+}
+
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(128) ns_embed_ngram_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, int64_t table_ld, float scale,
                                                              const T* __restrict__ bigram, int64_t bigram_ld, int64_t buckets, int64_t mul_prev,
                                                              int64_t mul_cur, const int32_t* __restrict__ slots, const int32_t* __restrict__ last,
@@ -35,6 +42,18 @@ __global__ void __launch_bounds__(128) ns_embed_ngram_kernel(const int32_t* __re
         g = bigram + bucket * bigram_ld;
     }
     float* out = y + (int64_t)row * dim;
+    if (VEC) {
+        for (int c = threadIdx.x * 4; c < dim; c += blockDim.x * 4) {
+            float4 v = embed_load4(t + c);
+            v = make_float4(__fmul_rn(v.x, scale), __fmul_rn(v.y, scale), __fmul_rn(v.z, scale), __fmul_rn(v.w, scale));
+            if (g != nullptr) {
+                const float4 r = embed_load4(g + c);
+                v = make_float4(__fadd_rn(v.x, r.x), __fadd_rn(v.y, r.y), __fadd_rn(v.z, r.z), __fadd_rn(v.w, r.w));
+            }
+            *reinterpret_cast<float4*>(out + c) = v;
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < dim; c += blockDim.x) {
         float v = __fmul_rn(ns_load(t + c), scale);
         if (g != nullptr) v = __fadd_rn(v, ns_load(g + c));
@@ -200,17 +219,16 @@ extern "C" int ns_embed_ngram(ns_device_t h, uint64_t ids, uint64_t table, int t
     NS_REQUIRE(float_or_bf16(table_dtype) && table_ld >= dim, NS_ERR_ARGUMENT, "ns_embed_ngram: bad table");
     NS_REQUIRE(bigram == 0 || (buckets > 0 && slots && last && bigram_ld >= dim), NS_ERR_ARGUMENT, "ns_embed_ngram: bad bigram table");
     const unsigned rows = (unsigned)batch * (unsigned)steps;
-    if (table_dtype == NS_F32)
-        NS_CUDA(ns_launch_plain(ns_embed_ngram_kernel<float>, dim3(rows), dim3(128), 0, d->stream, reinterpret_cast<const int32_t*>(ids),
-                                reinterpret_cast<const float*>(table), (int64_t)table_ld, scale, reinterpret_cast<const float*>(bigram), (int64_t)bigram_ld,
-                                (int64_t)buckets, mul_prev, mul_cur, reinterpret_cast<const int32_t*>(slots), reinterpret_cast<const int32_t*>(last), steps,
-                                dim, vocab, reinterpret_cast<float*>(y)));
-    else
-        NS_CUDA(ns_launch_plain(ns_embed_ngram_kernel<uint16_t>, dim3(rows), dim3(128), 0, d->stream, reinterpret_cast<const int32_t*>(ids),
-                                reinterpret_cast<const uint16_t*>(table), (int64_t)table_ld, scale, reinterpret_cast<const uint16_t*>(bigram),
-                                (int64_t)bigram_ld, (int64_t)buckets, mul_prev, mul_cur, reinterpret_cast<const int32_t*>(slots),
-                                reinterpret_cast<const int32_t*>(last), steps, dim, vocab, reinterpret_cast<float*>(y)));
-    return NS_OK;
+    const bool vec = ((dim | table_ld | (bigram ? bigram_ld : 0)) & 3) == 0 && ((table | bigram | y) & 15) == 0;
+    auto launch = [&](auto kernel, auto zero) -> int {
+        using T = decltype(zero);
+        NS_CUDA(ns_launch_plain(kernel, dim3(rows), dim3(128), 0, d->stream, reinterpret_cast<const int32_t*>(ids), reinterpret_cast<const T*>(table),
+                                (int64_t)table_ld, scale, reinterpret_cast<const T*>(bigram), (int64_t)bigram_ld, (int64_t)buckets, mul_prev, mul_cur,
+                                reinterpret_cast<const int32_t*>(slots), reinterpret_cast<const int32_t*>(last), steps, dim, vocab, reinterpret_cast<float*>(y)));
+        return NS_OK;
+    };
+    if (table_dtype == NS_F32) return vec ? launch(ns_embed_ngram_kernel<float, true>, float(0)) : launch(ns_embed_ngram_kernel<float, false>, float(0));
+    return vec ? launch(ns_embed_ngram_kernel<uint16_t, true>, uint16_t(0)) : launch(ns_embed_ngram_kernel<uint16_t, false>, uint16_t(0));
 }
 
 extern "C" int ns_rms_rows(ns_device_t h, uint64_t x, uint64_t src, int splits, int src_dtype, int src_ld, float alpha, uint64_t x_out, uint64_t w, float eps,

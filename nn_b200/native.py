@@ -99,6 +99,7 @@ SIGNATURES = {
     "ns_ids_from_f32": [vp, u64, u64, i32],
     "ns_short_conv": [vp, u64, i32, i32, i32, i32, P(i64), P(f32), i64, u64, u64, i32, i32, i32],
     "ns_delta_recurrent": [vp, u64, i32, u64, i32, u64, i32, u64, i32, i32, i32, u64, i32, i32, i32, u64, u64, i32, u64, i64, u64, i32, i32, i32, i32, i32, i32, u64, i32],
+    "ns_delta_chunked": [vp, u64, i32, u64, i32, u64, i32, u64, i32, i32, i32, u64, i32, i32, i32, u64, u64, i32, u64, i64, u64, i32, i32, i32, i32, i32, i32, u64, i32],
     "ns_gated_norm": [vp, u64, i32, u64, i32, i32, i32, i32, i32, u64, f32, i64, i32, i32, i32, u64, i32],
     "ns_latent_append": [vp, u64, i32, i32, i32, i32, i32, i32, i32, u64, u64, f32, u64, u64, u64, i32, i32, i32, u64, i32, u64, i64, i32, i32],
     "ns_rotate_heads": [vp, u64, i32, i32, i32, i32, i32, i32, i32, u64, u64, u64, i32, i32, i32, u64, i64, i32, i32, u64, i64, i32],

@@ -158,7 +158,7 @@ def test_short_convolution_over_cuts(dev, taps, cuts):
 
 
 # ------------------------------------------------------------------------------------------------ delta rule
-def run_delta(dev, data, cuts, H, kv, dim, vdim, channelwise, slots=(0,)):
+def run_delta(dev, data, cuts, H, kv, dim, vdim, channelwise, slots=(0,), chunk_from=1 << 30):
     """o [B, T, H, vdim] and final states, the sequences fed in `cuts`."""
     q, k, v, a, b, a_log, dt = data
     B, T = q.shape[:2]
@@ -173,7 +173,7 @@ def run_delta(dev, data, cuts, H, kv, dim, vdim, channelwise, slots=(0,)):
         dq, dk, dv = up(q), up(k), up(v)
         ab, ld = split_source(dev, np.concatenate([a[:, at:at + n].reshape(B * n, ac), b[:, at:at + n].reshape(B * n, H)], 1), 2)
         o = dev.empty(B * n * H * vdim)
-        N.call("ns_delta_recurrent", dev.handle, u(dq.ptr), kv * dim, u(dk.ptr), kv * dim, u(dv.ptr), H * vdim, u(ab.ptr), 2, ld, 0, u(ab.ptr), 2, ld, ac,
+        N.call("ns_delta_chunked" if n >= chunk_from else "ns_delta_recurrent", dev.handle, u(dq.ptr), kv * dim, u(dk.ptr), kv * dim, u(dv.ptr), H * vdim, u(ab.ptr), 2, ld, 0, u(ab.ptr), 2, ld, ac,
                u(da.ptr), u(dd.ptr), int(channelwise), u(state.ptr), i64(stride), u(st.slots.ptr), B, n, H, kv, dim, vdim, u(o.ptr), H * vdim)
         dev.synchronize()
         got[:, at:at + n] = o.download((B, n, H * vdim))
@@ -226,6 +226,43 @@ def test_delta_rule_over_cuts(dev, channelwise, cuts):
     eo, es = delta_oracle(data, channelwise)
     close(o, eo, 2e-5)
     close(s, es, 2e-5)
+
+
+@pytest.mark.parametrize("channelwise", [False, True])
+@pytest.mark.parametrize("T", [1, 16, 17, 63, 64, 65, 200])
+@pytest.mark.parametrize("H,kv,dim,vdim", [s for s in SIZES if s[2] <= 128] + [(2, 1, 33, 67)])
+def test_delta_rule_in_chunks(dev, H, kv, dim, vdim, T, channelwise):
+    data = delta_data(2, T, H, kv, dim, vdim, channelwise)
+    o, s = run_delta(dev, data, (T,), H, kv, dim, vdim, channelwise, slots=(2, 0), chunk_from=1)
+    eo, es = delta_oracle(data, channelwise)
+    close(o, eo, 1e-3)
+    close(s, es, 1e-3)
+
+
+@pytest.mark.parametrize("channelwise", [False, True])
+def test_chunks_and_single_tokens_carry_one_state(dev, channelwise):
+    cuts = (1, 40, 2, 64, 1, 1, 70)
+    data = delta_data(1, sum(cuts), 4, 2, 24, 48, channelwise)
+    o, s = run_delta(dev, data, cuts, 4, 2, 24, 48, channelwise, chunk_from=24)
+    eo, es = delta_oracle(data, channelwise)
+    close(o, eo, 1e-3)
+    close(s, es, 1e-3)
+
+
+@pytest.mark.parametrize("channelwise", [False, True])
+@pytest.mark.parametrize("kind", ["none", "total", "mixed"])
+def test_chunks_with_extreme_decays(dev, kind, channelwise):
+    """No decay at all, everything forgotten at every token, and both side by side: no exponent may overflow on the way."""
+    H, dim, vdim, T = 2, 64, 64, 130
+    q, k, v, a, b, a_log, dt = delta_data(1, T, H, 2, dim, vdim, channelwise)
+    rng = rng_for(13)
+    a = {"none": np.full_like(a, -60.0), "total": np.full_like(a, 60.0), "mixed": rng.choice([-60.0, 60.0, 0.0], a.shape)}[kind]
+    data = (q, k, v, a, b, np.full(H, 3.0), dt)
+    o, s = run_delta(dev, data, (T,), H, 2, dim, vdim, channelwise, chunk_from=1)
+    eo, es = delta_oracle(data, channelwise)
+    assert np.isfinite(o).all() and np.isfinite(s).all()
+    close(o, eo, 2e-3)
+    close(s, es, 2e-3)
 
 
 @pytest.mark.parametrize("act,name", [(N.ACT_SILU, "silu"), (N.ACT_SIGMOID, "sigmoid")])
