@@ -45,12 +45,43 @@ NS_DEVINL void split2(float x, float y, uint32_t& hi, uint32_t& lo)
     lo = ns_pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
 }
 NS_DEVINL void st32(uint32_t addr, uint32_t v) { asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
-// one accumulator += (hi + lo) (hi + lo) without the lo lo term
-NS_DEVINL void mma3(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1)
+// c[i][j] += (A_i hi + lo) (B_j hi + lo) without the lo lo term, for M row tiles and N pairs of column tiles.  One term after the other over
+// all accumulators, so that products which depend on one another are as far apart as the tile allows.
+template <int M, int N, int NC>
+NS_DEVINL void mma3(float (&c)[M][NC][4], int j0, const uint32_t (&ah)[M][4], const uint32_t (&al)[M][4], const uint32_t (&bh)[N][4], const uint32_t (&bl)[N][4])
 {
-    ns_mma_bf16(c, ah, bh0, bh1);
-    ns_mma_bf16(c, ah, bl0, bl1);
-    ns_mma_bf16(c, al, bh0, bh1);
+#pragma unroll
+    for (int term = 0; term < 3; term++)
+#pragma unroll
+        for (int j = 0; j < N; j++)
+#pragma unroll
+            for (int i = 0; i < M; i++)
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    const uint32_t(&x)[4] = term == 2 ? al[i] : ah[i];
+                    const uint32_t(&y)[4] = term == 1 ? bl[j] : bh[j];
+                    ns_mma_bf16(c[i][2 * (j0 + j) + h], x, y[2 * h], y[2 * h + 1]);
+                }
+}
+// four neighbouring channels of a row, zero beyond dim
+NS_DEVINL float4 row4(const float* p, int c, int dim, bool vec)
+{
+    if (vec) return c < dim ? *reinterpret_cast<const float4*>(p + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    return make_float4(c < dim ? p[c] : 0.0f, c + 1 < dim ? p[c + 1] : 0.0f, c + 2 < dim ? p[c + 2] : 0.0f, c + 3 < dim ? p[c + 3] : 0.0f);
+}
+NS_DEVINL float4 times(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+NS_DEVINL float4 exp2_of(float4 a, float4 b)      // 2^(a - b)
+{
+    return make_float4(ns_exp2(a.x - b.x), ns_exp2(a.y - b.y), ns_exp2(a.z - b.z), ns_exp2(a.w - b.w));
+}
+// four values as halves at `hi` and `lo`
+NS_DEVINL void st_split4(uint32_t hi, uint32_t lo, float4 v)
+{
+    uint32_t h0, l0, h1, l1;
+    split2(v.x, v.y, h0, l0);
+    split2(v.z, v.w, h1, l1);
+    asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(hi), "r"(h0), "r"(h1) : "memory");
+    asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(lo), "r"(l0), "r"(l1) : "memory");
 }
 
 template <int DK, int DV>
@@ -106,6 +137,8 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
     const float* qh = a.q + (int64_t)kvh * dim;
     const float* kh = a.k + (int64_t)kvh * dim;
     const float* vh = a.v + (int64_t)head * vdim + v0;
+    const bool vec = ((dim | a.q_ld | a.k_ld) & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k)) & 15) == 0;
+    const bool vec_a = CHANNEL && ((dim | a.a.ld | a.a_col) & 3) == 0 && (a.a.slab & 3) == 0 && (reinterpret_cast<uintptr_t>(a.a.ptr) & 15) == 0;
     const bool pair_v = ((a.v_ld | vdim | v0) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.v) & 7) == 0;
     const bool pair_o = ((a.o_ld | vdim | v0) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.o) & 7) == 0;
 
@@ -123,16 +156,26 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                 if (v0 + c < vdim && c < DV) asm volatile("prefetch.global.L2 [%0];" ::"l"(vh + (row0 + CH + r) * a.v_ld + c));
             }
         }
+        constexpr int QUADS = DK / 4;      // a thread takes four channels of a row
         // ------------------------------------------------------------ step sizes, running decays
         if (tid < CH) sBeta[tid] = tid < n ? ns_sigmoid(ns_source_at(a.b, (row0 + tid) * a.b.ld + a.b_col + head)) : 0.0f;
         if (CHANNEL) {
-            const int c = tid % DK;
-            const float dt = c < dim ? a.dt_bias[(int64_t)head * dim + c] : 0.0f;
+            const int c = (tid % QUADS) * 4;
+            const float4 dt = row4(a.dt_bias + (int64_t)head * dim, c, dim, false);
 #pragma unroll 4
-            for (int t = tid / DK; t < CH; t += 256 / DK)
-                sG[t * L::LG + c] = t < n && c < dim 
-                                         ? fmaxf(-rate2 * ns_softplus(ns_source_at(a.a, (row0 + t) * a.a.ld + a.a_col + head * dim + c) + dt), WEAKEST)
-                                         : 0.0f;
+            for (int t = tid / QUADS; t < CH; t += 256 / QUADS) {
+                float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (t < n && c < dim) {
+                    const int64_t at = (row0 + t) * a.a.ld + a.a_col + head * dim + c;
+                    if (vec_a) x = ns_source_at4(a.a, at);
+                    else
+                        x = make_float4(ns_source_at(a.a, at), c + 1 < dim ? ns_source_at(a.a, at + 1) : 0.0f, c + 2 < dim ? ns_source_at(a.a, at + 2) : 0.0f,
+                                        c + 3 < dim ? ns_source_at(a.a, at + 3) : 0.0f);
+                    x = make_float4(fmaxf(-rate2 * ns_softplus(x.x + dt.x), WEAKEST), fmaxf(-rate2 * ns_softplus(x.y + dt.y), WEAKEST),
+                                    fmaxf(-rate2 * ns_softplus(x.z + dt.z), WEAKEST), fmaxf(-rate2 * ns_softplus(x.w + dt.w), WEAKEST));
+                }
+                *reinterpret_cast<float4*>(sG + t * L::LG + c) = x;
+            }
             __syncthreads();
             if (tid < DK) {
                 float s = 0.0f;
@@ -160,51 +203,45 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
         __syncthreads();
 
         // ------------------------------------------------------------ A and P
-        // a thread takes two channels of a row
-        constexpr int PAIRS = DK / 2;
         if (!CHANNEL) {
             const float end = sGam[CH - 1];
-            for (int e = tid; e < CH * PAIRS; e += 256) {
-                const int t = e / PAIRS, c = (e % PAIRS) * 2;
-                float k0 = 0.0f, k1 = 0.0f, q0 = 0.0f, q1 = 0.0f;
+#pragma unroll 4
+            for (int e = tid; e < CH * QUADS; e += 256) {
+                const int t = e / QUADS, c = (e % QUADS) * 4;
+                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
                 if (t < n) {
-                    const float* kp = kh + (row0 + t) * a.k_ld;
-                    const float* qp = qh + (row0 + t) * a.q_ld;
-                    if (c < dim) { k0 = kp[c]; q0 = qp[c]; }
-                    if (c + 1 < dim) { k1 = kp[c + 1]; q1 = qp[c + 1]; }
+                    k4 = row4(kh + (row0 + t) * a.k_ld, c, dim, vec);
+                    q4 = row4(qh + (row0 + t) * a.q_ld, c, dim, vec);
                 }
                 const uint32_t at = base + (t * L::LK + c) * 2;
-                uint32_t hi, lo;
-                split2(k0, k1, hi, lo);
-                st32(at + L::KT, hi); st32(at + L::KT + L::KMAT, lo);
-                split2(q0, q1, hi, lo);
-                st32(at + L::QT, hi); st32(at + L::QT + L::KMAT, lo);
+                st_split4(at + L::KT, at + L::KT + L::KMAT, k4);
+                st_split4(at + L::QT, at + L::QT + L::KMAT, q4);
                 const float f = ns_exp2(end - sGam[t]);
-                split2(k0 * f, k1 * f, hi, lo);
-                st32(at + L::KB, hi); st32(at + L::KB + L::KMAT, lo);
+                st_split4(at + L::KB, at + L::KB + L::KMAT, make_float4(k4.x * f, k4.y * f, k4.z * f, k4.w * f));
             }
             __syncthreads();
             // warps 0..3: k rows, warps 4..7: q rows, 16 each, against all k
-            float acc[8][4];
+            float acc[1][8][4];
 #pragma unroll
             for (int j = 0; j < 8; j++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) acc[j][e] = 0.0f;
+                for (int e = 0; e < 4; e++) acc[0][j][e] = 0.0f;
             const uint32_t am = base + (warp < 4 ? L::KT : L::QT), bm = base + L::KT;
             const int mr = (warp & 3) * 16;
-#pragma unroll 2
+#pragma unroll 1
             for (int k = 0; k < DK; k += 16) {
-                uint32_t ah[4], al[4];
-                ns_ldsm4(ah, ns_addr_a(am, L::LK, mr, k, lane));
-                ns_ldsm4(al, ns_addr_a(am + L::KMAT, L::LK, mr, k, lane));
+                uint32_t ah[1][4], al[1][4], bh[2][4], bl[2][4];
+                ns_ldsm4(ah[0], ns_addr_a(am, L::LK, mr, k, lane));
+                ns_ldsm4(al[0], ns_addr_a(am + L::KMAT, L::LK, mr, k, lane));
 #pragma unroll
-                for (int j = 0; j < 4; j++) {
+                for (int j = 0; j < 4; j += 2) {
                     if (j * 16 > mr) continue;
-                    uint32_t bh[4], bl[4];
-                    ns_ldsm4(bh, ns_addr_b(bm, L::LK, j * 16, k, lane));
-                    ns_ldsm4(bl, ns_addr_b(bm + L::KMAT, L::LK, j * 16, k, lane));
-                    mma3(acc[2 * j], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                    mma3(acc[2 * j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+#pragma unroll
+                    for (int x = 0; x < 2; x++) {
+                        ns_ldsm4(bh[x], ns_addr_b(bm, L::LK, (j + x) * 16, k, lane));
+                        ns_ldsm4(bl[x], ns_addr_b(bm + L::KMAT, L::LK, (j + x) * 16, k, lane));
+                    }
+                    mma3(acc, j, ah, al, bh, bl);
                 }
             }
 #pragma unroll
@@ -213,41 +250,34 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                 for (int e = 0; e < 4; e++) {
                     const int r = mr + g + (e >> 1) * 8, c = j * 8 + t4 * 2 + (e & 1);
                     const float f = c <= r ? ns_exp2(sGam[r] - sGam[c]) : 0.0f;
-                    if (warp < 4) sA[r * L::LA + c] = c < r ? acc[j][e] * f * sBeta[r] : 0.0f;
-                    else sP[r * L::LA + c] = acc[j][e] * f;
+                    if (warp < 4) sA[r * L::LA + c] = c < r ? acc[0][j][e] * f * sBeta[r] : 0.0f;
+                    else sP[r * L::LA + c] = acc[0][j][e] * f;
                 }
             for (int c = tid; c < DK; c += 256) sEnd[c] = ns_exp2(end);
         } else {
             // rows of block I relative to the block's beginning (in KT, QT), columns before it likewise: block 1 in KB rows 0..15,
             // block 3 in KB rows 16..63, block 2 in the T area
-            for (int e = tid; e < CH * PAIRS; e += 256) {
-                const int t = e / PAIRS, c = (e % PAIRS) * 2, blk = t >> 4;
-                float k0 = 0.0f, k1 = 0.0f, q0 = 0.0f, q1 = 0.0f;
+#pragma unroll 2
+            for (int e = tid; e < CH * QUADS; e += 256) {
+                const int t = e / QUADS, c = (e % QUADS) * 4, blk = t >> 4;
+                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
                 if (t < n) {
-                    const float* kp = kh + (row0 + t) * a.k_ld;
-                    const float* qp = qh + (row0 + t) * a.q_ld;
-                    if (c < dim) { k0 = kp[c]; q0 = qp[c]; }
-                    if (c + 1 < dim) { k1 = kp[c + 1]; q1 = qp[c + 1]; }
+                    k4 = row4(kh + (row0 + t) * a.k_ld, c, dim, vec);
+                    q4 = row4(qh + (row0 + t) * a.q_ld, c, dim, vec);
                 }
-                const float2 G = *reinterpret_cast<const float2*>(sG + t * L::LG + c);
-                uint32_t hi, lo;
+                const float4 G = *reinterpret_cast<const float4*>(sG + t * L::LG + c);
                 if (blk > 0) {
-                    const float2 ref = *reinterpret_cast<const float2*>(sG + (blk * 16 - 1) * L::LG + c);
-                    const float f0 = ns_exp2(G.x - ref.x), f1 = ns_exp2(G.y - ref.y);
+                    const float4 f = exp2_of(G, *reinterpret_cast<const float4*>(sG + (blk * 16 - 1) * L::LG + c));
                     const uint32_t at = base + (t * L::LK + c) * 2;
-                    split2(k0 * f0, k1 * f1, hi, lo);
-                    st32(at + L::KT, hi); st32(at + L::KT + L::KMAT, lo);
-                    split2(q0 * f0, q1 * f1, hi, lo);
-                    st32(at + L::QT, hi); st32(at + L::QT + L::KMAT, lo);
+                    st_split4(at + L::KT, at + L::KT + L::KMAT, times(k4, f));
+                    st_split4(at + L::QT, at + L::QT + L::KMAT, times(q4, f));
                 }
 #pragma unroll
                 for (int I = 1; I < 4; I++) {
                     if (blk >= I) continue;
-                    const float2 ref = *reinterpret_cast<const float2*>(sG + (I * 16 - 1) * L::LG + c);
-                    split2(k0 * ns_exp2(ref.x - G.x), k1 * ns_exp2(ref.y - G.y), hi, lo);
+                    const float4 f = exp2_of(*reinterpret_cast<const float4*>(sG + (I * 16 - 1) * L::LG + c), G);
                     const uint32_t at = I == 2 ? base + L::T + (t * L::LK + c) * 2 : base + L::KB + (((I == 3 ? 16 : 0) + t) * L::LK + c) * 2;
-                    st32(at, hi);
-                    st32(at + (I == 2 ? 32 * L::LK * 2 : L::KMAT), lo);
+                    st_split4(at, at + (I == 2 ? 32 * L::LK * 2 : L::KMAT), times(k4, f));
                 }
             }
             __syncthreads();
@@ -257,25 +287,24 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                 const uint32_t am = base + (which ? L::QT : L::KT);
                 const uint32_t bh_m = I == 2 ? base + L::T : base + L::KB + (I == 3 ? 16 * L::LK * 2 : 0);
                 const uint32_t bl_m = bh_m + (I == 2 ? 32 * L::LK * 2 : L::KMAT);
-                float acc[6][4];
+                float acc[1][6][4];
 #pragma unroll
                 for (int j = 0; j < 6; j++)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) acc[j][e] = 0.0f;
-#pragma unroll 2
+                    for (int e = 0; e < 4; e++) acc[0][j][e] = 0.0f;
+#pragma unroll 1
                 for (int k = 0; k < DK; k += 16) {
-                    uint32_t ah[4], al[4];
-                    ns_ldsm4(ah, ns_addr_a(am, L::LK, I * 16, k, lane));
-                    ns_ldsm4(al, ns_addr_a(am + L::KMAT, L::LK, I * 16, k, lane));
+                    uint32_t ah[1][4], al[1][4], bh[3][4], bl[3][4];
+                    ns_ldsm4(ah[0], ns_addr_a(am, L::LK, I * 16, k, lane));
+                    ns_ldsm4(al[0], ns_addr_a(am + L::KMAT, L::LK, I * 16, k, lane));
 #pragma unroll
                     for (int j = 0; j < 3; j++) {
-                        if (j >= I) continue;
-                        uint32_t bh[4], bl[4];
-                        ns_ldsm4(bh, ns_addr_b(bh_m, L::LK, j * 16, k, lane));
-                        ns_ldsm4(bl, ns_addr_b(bl_m, L::LK, j * 16, k, lane));
-                        mma3(acc[2 * j], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                        mma3(acc[2 * j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                        // (blocks 1 and 2 multiply some rows that are not theirs; those columns are dropped below)
+                        const int n0 = j < I ? j * 16 : 0;
+                        ns_ldsm4(bh[j], ns_addr_b(bh_m, L::LK, n0, k, lane));
+                        ns_ldsm4(bl[j], ns_addr_b(bl_m, L::LK, n0, k, lane));
                     }
+                    mma3(acc, 0, ah, al, bh, bl);
                 }
 #pragma unroll
                 for (int j = 0; j < 6; j++)
@@ -283,8 +312,8 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                     for (int e = 0; e < 4; e++) {
                         const int r = I * 16 + g + (e >> 1) * 8, c = j * 8 + t4 * 2 + (e & 1);
                         if (c >= I * 16) continue;
-                        if (which) sP[r * L::LA + c] = acc[j][e];
-                        else sA[r * L::LA + c] = acc[j][e] * sBeta[r];
+                        if (which) sP[r * L::LA + c] = acc[0][j][e];
+                        else sA[r * L::LA + c] = acc[0][j][e] * sBeta[r];
                     }
             }
             // the 16 x 16 blocks on the diagonal, pair by pair: 16 lanes share a row, each a sixteenth of the channels
@@ -292,14 +321,19 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
             const int hl = lane & 15;
             for (int task = (warp + 2) & 7; task < CH / 2; task += 8) {
                 const int blk = task >> 3, ii = (lane >> 4) ? 15 - (task & 7) : (task & 7), i = blk * 16 + ii;
+                const int ch = hl * CPL;
                 float ki[CPL], qi[CPL], gi[CPL];
 #pragma unroll
-                for (int x = 0; x < CPL; x++) {
-                    const int c = hl * CPL + x;
-                    const bool in = i < n && c < dim;
-                    ki[x] = in ? kh[(row0 + i) * a.k_ld + c] : 0.0f;
-                    qi[x] = in ? qh[(row0 + i) * a.q_ld + c] : 0.0f;
-                    gi[x] = sG[i * L::LG + c];
+                for (int x = 0; x < CPL; x += 4) {
+                    float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
+                    if (i < n) {
+                        k4 = row4(kh + (row0 + i) * a.k_ld, ch + x, dim, vec);
+                        q4 = row4(qh + (row0 + i) * a.q_ld, ch + x, dim, vec);
+                    }
+                    const float4 G = *reinterpret_cast<const float4*>(sG + i * L::LG + ch + x);
+                    ki[x] = k4.x; ki[x + 1] = k4.y; ki[x + 2] = k4.z; ki[x + 3] = k4.w;
+                    qi[x] = q4.x; qi[x + 1] = q4.y; qi[x + 2] = q4.z; qi[x + 3] = q4.w;
+                    gi[x] = G.x; gi[x + 1] = G.y; gi[x + 2] = G.z; gi[x + 3] = G.w;
                 }
                 float v[32];
 #pragma unroll
@@ -307,12 +341,12 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                     float kk = 0.0f, qk = 0.0f;
                     if (j <= ii && blk * 16 + j < n) {
 #pragma unroll
-                        for (int x = 0; x < CPL; x++) {
-                            const int c = hl * CPL + x;
-                            const float kj = c < dim ? kh[(row0 + blk * 16 + j) * a.k_ld + c] : 0.0f;
-                            const float w = kj * ns_exp2(gi[x] - sG[(blk * 16 + j) * L::LG + c]);
-                            kk = fmaf(ki[x], w, kk);
-                            qk = fmaf(qi[x], w, qk);
+                        for (int x = 0; x < CPL; x += 4) {
+                            const float4 kj = row4(kh + (row0 + blk * 16 + j) * a.k_ld, ch + x, dim, vec);
+                            const float4 G = *reinterpret_cast<const float4*>(sG + (blk * 16 + j) * L::LG + ch + x);
+                            const float4 w = times(kj, exp2_of(make_float4(gi[x], gi[x + 1], gi[x + 2], gi[x + 3]), G));
+                            kk = fmaf(ki[x], w.x, fmaf(ki[x + 1], w.y, fmaf(ki[x + 2], w.z, fmaf(ki[x + 3], w.w, kk))));
+                            qk = fmaf(qi[x], w.x, fmaf(qi[x + 1], w.y, fmaf(qi[x + 2], w.z, fmaf(qi[x + 3], w.w, qk))));
                         }
                     }
                     v[j] = kk;
@@ -358,25 +392,19 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
 #pragma unroll
             for (int i = 0; i < 16; i++) blk[i * L::LA + col] = x[i];
         } else if (CHANNEL) {
-            for (int e = tid - 64; e < CH * PAIRS; e += 192) {
-                const int t = e / PAIRS, c = (e % PAIRS) * 2;
-                float k0 = 0.0f, k1 = 0.0f, q0 = 0.0f, q1 = 0.0f;
+#pragma unroll 2
+            for (int e = tid - 64; e < CH * QUADS; e += 192) {
+                const int t = e / QUADS, c = (e % QUADS) * 4;
+                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
                 if (t < n) {
-                    const float* kp = kh + (row0 + t) * a.k_ld;
-                    const float* qp = qh + (row0 + t) * a.q_ld;
-                    if (c < dim) { k0 = kp[c]; q0 = qp[c]; }
-                    if (c + 1 < dim) { k1 = kp[c + 1]; q1 = qp[c + 1]; }
+                    k4 = row4(kh + (row0 + t) * a.k_ld, c, dim, vec);
+                    q4 = row4(qh + (row0 + t) * a.q_ld, c, dim, vec);
                 }
-                const float2 G = *reinterpret_cast<const float2*>(sG + t * L::LG + c), end = *reinterpret_cast<const float2*>(sG + (CH - 1) * L::LG + c);
-                const float f0 = ns_exp2(G.x), f1 = ns_exp2(G.y);
+                const float4 G = *reinterpret_cast<const float4*>(sG + t * L::LG + c), f = exp2_of(G, make_float4(0.f, 0.f, 0.f, 0.f));
                 const uint32_t at = base + (t * L::LK + c) * 2;
-                uint32_t hi, lo;
-                split2(k0 * f0, k1 * f1, hi, lo);
-                st32(at + L::KT, hi); st32(at + L::KT + L::KMAT, lo);
-                split2(q0 * f0, q1 * f1, hi, lo);
-                st32(at + L::QT, hi); st32(at + L::QT + L::KMAT, lo);
-                split2(k0 * ns_exp2(end.x - G.x), k1 * ns_exp2(end.y - G.y), hi, lo);
-                st32(at + L::KB, hi); st32(at + L::KB + L::KMAT, lo);
+                st_split4(at + L::KT, at + L::KT + L::KMAT, times(k4, f));
+                st_split4(at + L::QT, at + L::QT + L::KMAT, times(q4, f));
+                st_split4(at + L::KB, at + L::KB + L::KMAT, times(k4, exp2_of(*reinterpret_cast<const float4*>(sG + (CH - 1) * L::LG + c), G)));
             }
         }
         __syncthreads();
@@ -476,15 +504,14 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                     ns_ldsm4(al[i], ns_addr_a(am + L::KMAT, L::LK, xr + i * 16, k, lane));
                 }
 #pragma unroll
-                for (int j = 0; j < NS / 2; j++) {
-                    uint32_t bh[4], bl[4];
-                    ns_ldsm4_t(bh, ns_addr_bt(bm, L::LV, k, sc0 + j * 16, lane));
-                    ns_ldsm4_t(bl, ns_addr_bt(bm + DK * L::LV * 2, L::LV, k, sc0 + j * 16, lane));
+                for (int j = 0; j < NS / 2; j += 2) {
+                    uint32_t bh[2][4], bl[2][4];
 #pragma unroll
-                    for (int i = 0; i < 2; i++) {
-                        mma3(acc[i][2 * j], ah[i], al[i], bh[0], bh[1], bl[0], bl[1]);
-                        mma3(acc[i][2 * j + 1], ah[i], al[i], bh[2], bh[3], bl[2], bl[3]);
+                    for (int x = 0; x < 2; x++) {
+                        ns_ldsm4_t(bh[x], ns_addr_bt(bm, L::LV, k, sc0 + (j + x) * 16, lane));
+                        ns_ldsm4_t(bl[x], ns_addr_bt(bm + DK * L::LV * 2, L::LV, k, sc0 + (j + x) * 16, lane));
                     }
+                    mma3(acc, j, ah, al, bh, bl);
                 }
             }
         }
@@ -538,17 +565,13 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                     ns_ldsm4(ah[i], ns_addr_a(base + L::T, L::LT, ur + i * 16, k, lane));
                     ns_ldsm4(al[i], ns_addr_a(base + L::T + L::TMAT, L::LT, ur + i * 16, k, lane));
                 }
+                uint32_t bh[NU / 2][4], bl[NU / 2][4];
 #pragma unroll
                 for (int j = 0; j < NU / 2; j++) {
-                    uint32_t bh[4], bl[4];
-                    ns_ldsm4_t(bh, ns_addr_bt(base + L::U, L::LV, k, uc + j * 16, lane));
-                    ns_ldsm4_t(bl, ns_addr_bt(base + L::U + L::VMAT, L::LV, k, uc + j * 16, lane));
-#pragma unroll
-                    for (int i = 0; i < 2; i++) {
-                        mma3(ua[i][2 * j], ah[i], al[i], bh[0], bh[1], bl[0], bl[1]);
-                        mma3(ua[i][2 * j + 1], ah[i], al[i], bh[2], bh[3], bl[2], bl[3]);
-                    }
+                    ns_ldsm4_t(bh[j], ns_addr_bt(base + L::U, L::LV, k, uc + j * 16, lane));
+                    ns_ldsm4_t(bl[j], ns_addr_bt(base + L::U + L::VMAT, L::LV, k, uc + j * 16, lane));
                 }
+                mma3(ua, 0, ah, al, bh, bl);
             }
             __syncthreads();
 #pragma unroll
@@ -593,15 +616,14 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                     ns_ldsm4(al[i], ns_addr_a(base + L::T + L::TMAT, L::LT, xr + i * 16, k, lane));
                 }
 #pragma unroll
-                for (int j = 0; j < NS / 2; j++) {
-                    uint32_t bh[4], bl[4];
-                    ns_ldsm4_t(bh, ns_addr_bt(base + L::U, L::LV, k, sc0 + j * 16, lane));
-                    ns_ldsm4_t(bl, ns_addr_bt(base + L::U + L::VMAT, L::LV, k, sc0 + j * 16, lane));
+                for (int j = 0; j < NS / 2; j += 2) {
+                    uint32_t bh[2][4], bl[2][4];
 #pragma unroll
-                    for (int i = 0; i < 2; i++) {
-                        mma3(acc[i][2 * j], ah[i], al[i], bh[0], bh[1], bl[0], bl[1]);
-                        mma3(acc[i][2 * j + 1], ah[i], al[i], bh[2], bh[3], bl[2], bl[3]);
+                    for (int x = 0; x < 2; x++) {
+                        ns_ldsm4_t(bh[x], ns_addr_bt(base + L::U, L::LV, k, sc0 + (j + x) * 16, lane));
+                        ns_ldsm4_t(bl[x], ns_addr_bt(base + L::U + L::VMAT, L::LV, k, sc0 + (j + x) * 16, lane));
                     }
+                    mma3(acc, j, ah, al, bh, bl);
                 }
             }
 #pragma unroll
@@ -641,15 +663,14 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
                 ns_ldsm4_t(al[i], ns_addr_at(base + L::KB + L::KMAT, L::LK, sr0 + i * 16, k, lane));
             }
 #pragma unroll
-            for (int j = 0; j < NS / 2; j++) {
-                uint32_t bh[4], bl[4];
-                ns_ldsm4_t(bh, ns_addr_bt(base + L::U, L::LV, k, sc0 + j * 16, lane));
-                ns_ldsm4_t(bl, ns_addr_bt(base + L::U + L::VMAT, L::LV, k, sc0 + j * 16, lane));
+            for (int j = 0; j < NS / 2; j += 2) {
+                uint32_t bh[2][4], bl[2][4];
 #pragma unroll
-                for (int i = 0; i < MS; i++) {
-                    mma3(st[i][2 * j], ah[i], al[i], bh[0], bh[1], bl[0], bl[1]);
-                    mma3(st[i][2 * j + 1], ah[i], al[i], bh[2], bh[3], bl[2], bl[3]);
+                for (int x = 0; x < 2; x++) {
+                    ns_ldsm4_t(bh[x], ns_addr_bt(base + L::U, L::LV, k, sc0 + (j + x) * 16, lane));
+                    ns_ldsm4_t(bl[x], ns_addr_bt(base + L::U + L::VMAT, L::LV, k, sc0 + (j + x) * 16, lane));
                 }
+                mma3(st, j, ah, al, bh, bl);
             }
         }
         __syncthreads();
