@@ -454,7 +454,7 @@ NS_API int ns_delta_recurrent(ns_device_t dev, uint64_t q, int q_ld, uint64_t k,
                               uint64_t state, int64_t state_slot_stride, uint64_t slots, int batch, int steps, int heads, int kv_heads, int dim, int vdim,
                               uint64_t o, int o_ld);
 /* The same for a prompt's portion, 64 tokens at a time on the tensor cores (bf16 halves of 32-bit operands, three products each:
- * about 16 mantissa bits; state and sums 32-bit).  dim <= 128. */
+ * about 16 mantissa bits; state and sums 32-bit).  dim <= 128 and a multiple of 4, vdim even, rows 16-byte (v, o: 8-byte) aligned. */
 NS_API int ns_delta_chunked(ns_device_t dev, uint64_t q, int q_ld, uint64_t k, int k_ld, uint64_t v, int v_ld, uint64_t a_src, int a_splits, int a_ld,
                             int a_col, uint64_t b_src, int b_splits, int b_ld, int b_col, uint64_t a_log, uint64_t dt_bias, int per_channel,
                             uint64_t state, int64_t state_slot_stride, uint64_t slots, int batch, int steps, int heads, int kv_heads, int dim, int vdim,

@@ -200,7 +200,7 @@ class DeltaMixer:
         self.dev, self.ws, self.eps = ws.dev, ws, eps
         self.heads, self.kv_heads, self.dim, self.vdim, self.taps = heads, kv_heads, dim, vdim, taps
         self.channelwise = "a1" in w
-        self.chunks = ws.dtype == N.NS_BF16 and dim <= 128
+        self.chunks = ws.dtype == N.NS_BF16 and dim <= 128 and dim % 4 == 0 and vdim % 2 == 0
         dev = self.dev
         up = lambda a: dev.from_numpy(f32(a).reshape(-1))
         self.conv = [up(w[n + "_conv"]) for n in "qkv"]

@@ -64,11 +64,7 @@ NS_DEVINL void mma3(float (&c)[M][NC][4], int j0, const uint32_t (&ah)[M][4], co
                 }
 }
 // four neighbouring channels of a row, zero beyond dim
-NS_DEVINL float4 row4(const float* p, int c, int dim, bool vec)
-{
-    if (vec) return c < dim ? *reinterpret_cast<const float4*>(p + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-    return make_float4(c < dim ? p[c] : 0.0f, c + 1 < dim ? p[c + 1] : 0.0f, c + 2 < dim ? p[c + 2] : 0.0f, c + 3 < dim ? p[c + 3] : 0.0f);
-}
+NS_DEVINL float4 row4(const float* p, int c, int dim) { return c < dim ? *reinterpret_cast<const float4*>(p + c) : make_float4(0.f, 0.f, 0.f, 0.f); }
 NS_DEVINL float4 times(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 NS_DEVINL float4 exp2_of(float4 a, float4 b)      // 2^(a - b)
 {
@@ -84,11 +80,21 @@ NS_DEVINL void st_split4(uint32_t hi, uint32_t lo, float4 v)
     asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(lo), "r"(l0), "r"(l1) : "memory");
 }
 
+// log(1 + e^z) in 32-bit: the logarithm where 1 + e holds e's digits, its series below
+NS_DEVINL float softplus(float z)
+{
+    const float e = ns_exp2(-fabsf(z) * LOG2E);
+    const float l = e < 0.015625f ? e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333333f), -0.5f), 1.0f) : logf(1.0f + e);
+    return fmaxf(z, 0.0f) + l;
+}
+
 template <int DK, int DV>
 struct ChunkSmem {
     static constexpr int LK = DK + 8, LV = DV + 8, LT = CH + 8, LG = DK + 4, LA = CH + 1;
     static constexpr int KMAT = CH * LK * 2, VMAT = CH * LV * 2, TMAT = CH * LT * 2;      // bytes of one half
-    static constexpr int KT = 0, QT = KT + 2 * KMAT, KB = QT + 2 * KMAT, U = KB + 2 * KMAT, T = U + 2 * VMAT, X = T + 2 * TMAT;
+    // U also holds the keys as they are while A and P are made
+    static constexpr int U_BYTES = 2 * VMAT > CH * LG * 4 ? 2 * VMAT : CH * LG * 4;
+    static constexpr int KT = 0, QT = KT + 2 * KMAT, KB = QT + 2 * KMAT, U = KB + 2 * KMAT, T = U + U_BYTES, X = T + 2 * TMAT;
     static constexpr int S_BYTES = 2 * DK * LV * 2, G_BYTES = CH * LG * 4, A_BYTES = CH * LA * 4;
     static constexpr int X_BYTES = S_BYTES > G_BYTES + 2 * A_BYTES ? S_BYTES : G_BYTES + 2 * A_BYTES;
     static constexpr int SMALL = X + X_BYTES;                                              // beta, gamma, end decay
@@ -108,6 +114,7 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
     float* sA = reinterpret_cast<float*>(ch_smem + L::X + L::G_BYTES);          // A, then its inverse
     float* sP = sA + CH * L::LA;
     float* sW = reinterpret_cast<float*>(ch_smem + L::U);
+    float* sK = sW;
     float* sBeta = reinterpret_cast<float*>(ch_smem + L::SMALL);
     float* sGam = sBeta + CH;                                                   // running log2 decay per token (scalar mode)
     float* sEnd = sGam + CH;                                                    // decay of a state row over the chunk
@@ -137,10 +144,6 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
     const float* qh = a.q + (int64_t)kvh * dim;
     const float* kh = a.k + (int64_t)kvh * dim;
     const float* vh = a.v + (int64_t)head * vdim + v0;
-    const bool vec = ((dim | a.q_ld | a.k_ld) & 3) == 0 && ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k)) & 15) == 0;
-    const bool vec_a = CHANNEL && ((dim | a.a.ld | a.a_col) & 3) == 0 && (a.a.slab & 3) == 0 && (reinterpret_cast<uintptr_t>(a.a.ptr) & 15) == 0;
-    const bool pair_v = ((a.v_ld | vdim | v0) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.v) & 7) == 0;
-    const bool pair_o = ((a.o_ld | vdim | v0) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.o) & 7) == 0;
 
     for (int c0 = 0; c0 < a.steps; c0 += CH) {
         const int n = min(CH, a.steps - c0);
@@ -157,22 +160,31 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
             }
         }
         constexpr int QUADS = DK / 4;      // a thread takes four channels of a row
+        // keys and queries of elements e0, e0 + stride, ... (four of them), all loaded before the caller stores any
+        auto load_rows = [&](int e0, int stride, float4 (&k4)[4], float4 (&q4)[4]) {
+#pragma unroll
+            for (int x = 0; x < 4; x++) {
+                const int e = e0 + stride * x, t = e / QUADS, c = (e % QUADS) * 4;
+                k4[x] = q4[x] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (t < n) {
+                    k4[x] = row4(kh + (row0 + t) * a.k_ld, c, dim);
+                    q4[x] = row4(qh + (row0 + t) * a.q_ld, c, dim);
+                }
+            }
+        };
         // ------------------------------------------------------------ step sizes, running decays
         if (tid < CH) sBeta[tid] = tid < n ? ns_sigmoid(ns_source_at(a.b, (row0 + tid) * a.b.ld + a.b_col + head)) : 0.0f;
         if (CHANNEL) {
             const int c = (tid % QUADS) * 4;
-            const float4 dt = row4(a.dt_bias + (int64_t)head * dim, c, dim, false);
-#pragma unroll 4
+            const float4 dt = row4(a.dt_bias + (int64_t)head * dim, c, dim);
+#pragma unroll 8
             for (int t = tid / QUADS; t < CH; t += 256 / QUADS) {
                 float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
                 if (t < n && c < dim) {
                     const int64_t at = (row0 + t) * a.a.ld + a.a_col + head * dim + c;
-                    if (vec_a) x = ns_source_at4(a.a, at);
-                    else
-                        x = make_float4(ns_source_at(a.a, at), c + 1 < dim ? ns_source_at(a.a, at + 1) : 0.0f, c + 2 < dim ? ns_source_at(a.a, at + 2) : 0.0f,
-                                        c + 3 < dim ? ns_source_at(a.a, at + 3) : 0.0f);
-                    x = make_float4(fmaxf(-rate2 * ns_softplus(x.x + dt.x), WEAKEST), fmaxf(-rate2 * ns_softplus(x.y + dt.y), WEAKEST),
-                                    fmaxf(-rate2 * ns_softplus(x.z + dt.z), WEAKEST), fmaxf(-rate2 * ns_softplus(x.w + dt.w), WEAKEST));
+                    x = ns_source_at4(a.a, at);
+                    x = make_float4(fmaxf(-rate2 * softplus(x.x + dt.x), WEAKEST), fmaxf(-rate2 * softplus(x.y + dt.y), WEAKEST),
+                                    fmaxf(-rate2 * softplus(x.z + dt.z), WEAKEST), fmaxf(-rate2 * softplus(x.w + dt.w), WEAKEST));
                 }
                 *reinterpret_cast<float4*>(sG + t * L::LG + c) = x;
             }
@@ -189,7 +201,7 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
 #pragma unroll
             for (int i = 0; i < 2; i++) {
                 const int t = 2 * lane + i;
-                x[i] = t < n ? fmaxf(-rate2 * ns_softplus(ns_source_at(a.a, (row0 + t) * a.a.ld + a.a_col + head) + dt), WEAKEST) : 0.0f;
+                x[i] = t < n ? fmaxf(-rate2 * softplus(ns_source_at(a.a, (row0 + t) * a.a.ld + a.a_col + head) + dt), WEAKEST) : 0.0f;
             }
             float s = x[0] + x[1];
 #pragma unroll
@@ -205,19 +217,18 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
         // ------------------------------------------------------------ A and P
         if (!CHANNEL) {
             const float end = sGam[CH - 1];
-#pragma unroll 4
-            for (int e = tid; e < CH * QUADS; e += 256) {
-                const int t = e / QUADS, c = (e % QUADS) * 4;
-                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
-                if (t < n) {
-                    k4 = row4(kh + (row0 + t) * a.k_ld, c, dim, vec);
-                    q4 = row4(qh + (row0 + t) * a.q_ld, c, dim, vec);
+            for (int e0 = tid; e0 < CH * QUADS; e0 += 1024) {
+                float4 k4[4], q4[4];
+                load_rows(e0, 256, k4, q4);
+#pragma unroll
+                for (int x = 0; x < 4; x++) {
+                    const int e = e0 + 256 * x, t = e / QUADS, c = (e % QUADS) * 4;
+                    const uint32_t at = base + (t * L::LK + c) * 2;
+                    st_split4(at + L::KT, at + L::KT + L::KMAT, k4[x]);
+                    st_split4(at + L::QT, at + L::QT + L::KMAT, q4[x]);
+                    const float f = ns_exp2(end - sGam[t]);
+                    st_split4(at + L::KB, at + L::KB + L::KMAT, make_float4(k4[x].x * f, k4[x].y * f, k4[x].z * f, k4[x].w * f));
                 }
-                const uint32_t at = base + (t * L::LK + c) * 2;
-                st_split4(at + L::KT, at + L::KT + L::KMAT, k4);
-                st_split4(at + L::QT, at + L::QT + L::KMAT, q4);
-                const float f = ns_exp2(end - sGam[t]);
-                st_split4(at + L::KB, at + L::KB + L::KMAT, make_float4(k4.x * f, k4.y * f, k4.z * f, k4.w * f));
             }
             __syncthreads();
             // warps 0..3: k rows, warps 4..7: q rows, 16 each, against all k
@@ -257,27 +268,27 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
         } else {
             // rows of block I relative to the block's beginning (in KT, QT), columns before it likewise: block 1 in KB rows 0..15,
             // block 3 in KB rows 16..63, block 2 in the T area
-#pragma unroll 2
-            for (int e = tid; e < CH * QUADS; e += 256) {
-                const int t = e / QUADS, c = (e % QUADS) * 4, blk = t >> 4;
-                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
-                if (t < n) {
-                    k4 = row4(kh + (row0 + t) * a.k_ld, c, dim, vec);
-                    q4 = row4(qh + (row0 + t) * a.q_ld, c, dim, vec);
-                }
-                const float4 G = *reinterpret_cast<const float4*>(sG + t * L::LG + c);
-                if (blk > 0) {
-                    const float4 f = exp2_of(G, *reinterpret_cast<const float4*>(sG + (blk * 16 - 1) * L::LG + c));
-                    const uint32_t at = base + (t * L::LK + c) * 2;
-                    st_split4(at + L::KT, at + L::KT + L::KMAT, times(k4, f));
-                    st_split4(at + L::QT, at + L::QT + L::KMAT, times(q4, f));
-                }
+            for (int e0 = tid; e0 < CH * QUADS; e0 += 1024) {
+                float4 k4[4], q4[4];
+                load_rows(e0, 256, k4, q4);
 #pragma unroll
-                for (int I = 1; I < 4; I++) {
-                    if (blk >= I) continue;
-                    const float4 f = exp2_of(*reinterpret_cast<const float4*>(sG + (I * 16 - 1) * L::LG + c), G);
-                    const uint32_t at = I == 2 ? base + L::T + (t * L::LK + c) * 2 : base + L::KB + (((I == 3 ? 16 : 0) + t) * L::LK + c) * 2;
-                    st_split4(at, at + (I == 2 ? 32 * L::LK * 2 : L::KMAT), times(k4, f));
+                for (int x = 0; x < 4; x++) {
+                    const int e = e0 + 256 * x, t = e / QUADS, c = (e % QUADS) * 4, blk = t >> 4;
+                    const float4 G = *reinterpret_cast<const float4*>(sG + t * L::LG + c);
+                    *reinterpret_cast<float4*>(sK + t * L::LG + c) = k4[x];
+                    if (blk > 0) {
+                        const float4 f = exp2_of(G, *reinterpret_cast<const float4*>(sG + (blk * 16 - 1) * L::LG + c));
+                        const uint32_t at = base + (t * L::LK + c) * 2;
+                        st_split4(at + L::KT, at + L::KT + L::KMAT, times(k4[x], f));
+                        st_split4(at + L::QT, at + L::QT + L::KMAT, times(q4[x], f));
+                    }
+#pragma unroll
+                    for (int I = 1; I < 4; I++) {
+                        if (blk >= I) continue;
+                        const float4 f = exp2_of(*reinterpret_cast<const float4*>(sG + (I * 16 - 1) * L::LG + c), G);
+                        const uint32_t at = I == 2 ? base + L::T + (t * L::LK + c) * 2 : base + L::KB + (((I == 3 ? 16 : 0) + t) * L::LK + c) * 2;
+                        st_split4(at, at + (I == 2 ? 32 * L::LK * 2 : L::KMAT), times(k4[x], f));
+                    }
                 }
             }
             __syncthreads();
@@ -321,54 +332,56 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
             const int hl = lane & 15;
             for (int task = (warp + 2) & 7; task < CH / 2; task += 8) {
                 const int blk = task >> 3, ii = (lane >> 4) ? 15 - (task & 7) : (task & 7), i = blk * 16 + ii;
-                const int ch = hl * CPL;
+                const int ch = hl * 4;      // channels ch + 64 y: 16 lanes read 256 neighbouring bytes
                 float ki[CPL], qi[CPL], gi[CPL];
 #pragma unroll
                 for (int x = 0; x < CPL; x += 4) {
-                    float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
-                    if (i < n) {
-                        k4 = row4(kh + (row0 + i) * a.k_ld, ch + x, dim, vec);
-                        q4 = row4(qh + (row0 + i) * a.q_ld, ch + x, dim, vec);
-                    }
-                    const float4 G = *reinterpret_cast<const float4*>(sG + i * L::LG + ch + x);
+                    const float4 k4 = *reinterpret_cast<const float4*>(sK + i * L::LG + ch + 16 * x);
+                    const float4 q4 = i < n ? row4(qh + (row0 + i) * a.q_ld, ch + 16 * x, dim) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float4 G = *reinterpret_cast<const float4*>(sG + i * L::LG + ch + 16 * x);
                     ki[x] = k4.x; ki[x + 1] = k4.y; ki[x + 2] = k4.z; ki[x + 3] = k4.w;
                     qi[x] = q4.x; qi[x + 1] = q4.y; qi[x + 2] = q4.z; qi[x + 3] = q4.w;
                     gi[x] = G.x; gi[x + 1] = G.y; gi[x + 2] = G.z; gi[x + 3] = G.w;
                 }
-                float v[32];
+                // columns in groups of four; what lies right of the diagonal is dropped afterwards
+                const int groups = (max(task & 7, 15 - (task & 7)) >> 2) + 1;
+#pragma unroll 1
+                for (int j0 = 0; j0 < groups * 4; j0 += 4) {
+                    const int t0 = blk * 16 + j0;
+                    float v[8];
 #pragma unroll
-                for (int j = 0; j < 16; j++) {
-                    float kk = 0.0f, qk = 0.0f;
-                    if (j <= ii && blk * 16 + j < n) {
+                    for (int x = 0; x < 4; x++) {
+                        float kk = 0.0f, qk = 0.0f;
 #pragma unroll
-                        for (int x = 0; x < CPL; x += 4) {
-                            const float4 kj = row4(kh + (row0 + blk * 16 + j) * a.k_ld, ch + x, dim, vec);
-                            const float4 G = *reinterpret_cast<const float4*>(sG + (blk * 16 + j) * L::LG + ch + x);
-                            const float4 w = times(kj, exp2_of(make_float4(gi[x], gi[x + 1], gi[x + 2], gi[x + 3]), G));
-                            kk = fmaf(ki[x], w.x, fmaf(ki[x + 1], w.y, fmaf(ki[x + 2], w.z, fmaf(ki[x + 3], w.w, kk))));
-                            qk = fmaf(qi[x], w.x, fmaf(qi[x + 1], w.y, fmaf(qi[x + 2], w.z, fmaf(qi[x + 3], w.w, qk))));
+                        for (int y = 0; y < CPL / 4; y++) {
+                            const float4 G = *reinterpret_cast<const float4*>(sG + (t0 + x) * L::LG + ch + 64 * y);
+                            const float4 k4 = *reinterpret_cast<const float4*>(sK + (t0 + x) * L::LG + ch + 64 * y);
+                            const float w0 = k4.x * ns_exp2(fminf(gi[4 * y] - G.x, 0.0f)), w1 = k4.y * ns_exp2(fminf(gi[4 * y + 1] - G.y, 0.0f));
+                            const float w2 = k4.z * ns_exp2(fminf(gi[4 * y + 2] - G.z, 0.0f)), w3 = k4.w * ns_exp2(fminf(gi[4 * y + 3] - G.w, 0.0f));
+                            kk = fmaf(ki[4 * y], w0, fmaf(ki[4 * y + 1], w1, fmaf(ki[4 * y + 2], w2, fmaf(ki[4 * y + 3], w3, kk))));
+                            qk = fmaf(qi[4 * y], w0, fmaf(qi[4 * y + 1], w1, fmaf(qi[4 * y + 2], w2, fmaf(qi[4 * y + 3], w3, qk))));
+                        }
+                        v[x] = kk;
+                        v[4 + x] = qk;
+                    }
+                    // sums over the 16 lanes; two lanes end up with the same one of the eight values
+#pragma unroll
+                    for (int m = 8, half = 4; m >= 2; m >>= 1, half >>= 1) {
+                        const bool up = (lane & m) != 0;
+#pragma unroll
+                        for (int x = 0; x < half; x++) {
+                            const float give = up ? v[x] : v[x + half], keep = up ? v[x + half] : v[x];
+                            v[x] = keep + __shfl_xor_sync(0xffffffffu, give, m);
                         }
                     }
-                    v[j] = kk;
-                    v[16 + j] = qk;
-                }
-                // sums over the 16 lanes, two of the 32 values ending up in each
-#pragma unroll
-                for (int m = 8, half = 16; m >= 1; m >>= 1, half >>= 1) {
-                    const bool up = (lane & m) != 0;
-#pragma unroll
-                    for (int x = 0; x < half; x++) {
-                        const float give = up ? v[x] : v[x + half], keep = up ? v[x + half] : v[x];
-                        v[x] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+                    v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+                    const int j = j0 + ((lane >> 1) & 1) + ((lane >> 1) & 2);
+                    if ((lane & 1) == 0) {
+                        if (lane & 8) sP[i * L::LA + blk * 16 + j] = j <= ii ? v[0] : 0.0f;
+                        else sA[i * L::LA + blk * 16 + j] = j < ii ? v[0] * sBeta[i] : 0.0f;
                     }
                 }
-                const int first = ((lane & 8) ? 16 : 0) + ((lane & 4) ? 8 : 0) + ((lane & 2) ? 4 : 0) + ((lane & 1) ? 2 : 0);
-#pragma unroll
-                for (int x = 0; x < 2; x++) {
-                    const int idx = first + x, j = idx & 15;
-                    if (idx < 16) sA[i * L::LA + blk * 16 + j] = j < ii ? v[x] * sBeta[i] : 0.0f;
-                    else sP[i * L::LA + blk * 16 + j] = j <= ii ? v[x] : 0.0f;
-                }
+                for (int j = groups * 4 + hl; j < 16; j += 16) sA[i * L::LA + blk * 16 + j] = sP[i * L::LA + blk * 16 + j] = 0.0f;
                 // right of the diagonal block
                 for (int c = (blk + 1) * 16 + hl; c < CH; c += 16) sA[i * L::LA + c] = sP[i * L::LA + c] = 0.0f;
             }
@@ -392,19 +405,19 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
 #pragma unroll
             for (int i = 0; i < 16; i++) blk[i * L::LA + col] = x[i];
         } else if (CHANNEL) {
-#pragma unroll 2
-            for (int e = tid - 64; e < CH * QUADS; e += 192) {
-                const int t = e / QUADS, c = (e % QUADS) * 4;
-                float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
-                if (t < n) {
-                    k4 = row4(kh + (row0 + t) * a.k_ld, c, dim, vec);
-                    q4 = row4(qh + (row0 + t) * a.q_ld, c, dim, vec);
+            for (int e0 = tid - 64; e0 < CH * QUADS; e0 += 768) {
+                float4 k4[4], q4[4];
+                load_rows(e0, 192, k4, q4);
+#pragma unroll
+                for (int x = 0; x < 4; x++) {
+                    const int e = e0 + 192 * x, t = e / QUADS, c = (e % QUADS) * 4;
+                    if (e >= CH * QUADS) break;
+                    const float4 G = *reinterpret_cast<const float4*>(sG + t * L::LG + c), f = exp2_of(G, make_float4(0.f, 0.f, 0.f, 0.f));
+                    const uint32_t at = base + (t * L::LK + c) * 2;
+                    st_split4(at + L::KT, at + L::KT + L::KMAT, times(k4[x], f));
+                    st_split4(at + L::QT, at + L::QT + L::KMAT, times(q4[x], f));
+                    st_split4(at + L::KB, at + L::KB + L::KMAT, times(k4[x], exp2_of(*reinterpret_cast<const float4*>(sG + (CH - 1) * L::LG + c), G)));
                 }
-                const float4 G = *reinterpret_cast<const float4*>(sG + t * L::LG + c), f = exp2_of(G, make_float4(0.f, 0.f, 0.f, 0.f));
-                const uint32_t at = base + (t * L::LK + c) * 2;
-                st_split4(at + L::KT, at + L::KT + L::KMAT, times(k4, f));
-                st_split4(at + L::QT, at + L::QT + L::KMAT, times(q4, f));
-                st_split4(at + L::KB, at + L::KB + L::KMAT, times(k4, exp2_of(*reinterpret_cast<const float4*>(sG + (CH - 1) * L::LG + c), G)));
             }
         }
         __syncthreads();
@@ -516,33 +529,35 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
             }
         }
         if (kside) {
-            // right-hand side beta (v - decayed read)
+            // right-hand side beta (v - decayed read); the values of 16 rows are loaded before any is used
 #pragma unroll
-            for (int i = 0; i < 2; i++)
+            for (int i = 0; i < 2; i++) {
+                float2 y[2][NS];
 #pragma unroll
                 for (int h = 0; h < 2; h++) {
                     const int r = xr + i * 16 + g + h * 8;
-                    const float beta = sBeta[r], f = CHANNEL ? 1.0f : ns_exp2(sGam[r]);
                     const float* vp = vh + (row0 + r) * a.v_ld;
 #pragma unroll
                     for (int j = 0; j < NS; j++) {
                         const int c = sc0 + j * 8 + t4 * 2;
-                        float y0 = 0.0f, y1 = 0.0f;
-                        if (r < n) {
-                            if (pair_v && v0 + c + 1 < vdim) {
-                                const float2 t = *reinterpret_cast<const float2*>(vp + c);
-                                y0 = t.x; y1 = t.y;
-                            } else {
-                                if (v0 + c < vdim) y0 = vp[c];
-                                if (v0 + c + 1 < vdim) y1 = vp[c + 1];
-                            }
-                        }
+                        y[h][j] = make_float2(0.0f, 0.0f);
+                        if (r >= n) continue;
+                        if (v0 + c < vdim) y[h][j] = *reinterpret_cast<const float2*>(vp + c);
+                    }
+                }
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    const int r = xr + i * 16 + g + h * 8;
+                    const float beta = sBeta[r], f = CHANNEL ? 1.0f : ns_exp2(sGam[r]);
+#pragma unroll
+                    for (int j = 0; j < NS; j++) {
                         uint32_t hi, lo;
-                        split2(beta * fmaf(-f, acc[i][j][2 * h], y0), beta * fmaf(-f, acc[i][j][2 * h + 1], y1), hi, lo);
-                        const uint32_t at = base + L::U + (r * L::LV + c) * 2;
+                        split2(beta * fmaf(-f, acc[i][j][2 * h], y[h][j].x), beta * fmaf(-f, acc[i][j][2 * h + 1], y[h][j].y), hi, lo);
+                        const uint32_t at = base + L::U + (r * L::LV + sc0 + j * 8 + t4 * 2) * 2;
                         st32(at, hi); st32(at + L::VMAT, lo);
                     }
                 }
+            }
         }
         __syncthreads();
         // ------------------------------------------------------------ U = T (right-hand side)
@@ -636,12 +651,7 @@ __global__ void __launch_bounds__(256, 1) ns_delta_chunk_kernel(const ChunkArgs 
 #pragma unroll
                     for (int j = 0; j < NS; j++) {
                         const int c = sc0 + j * 8 + t4 * 2;
-                        if (pair_o && v0 + c + 1 < vdim) {
-                            *reinterpret_cast<float2*>(op + c) = make_float2(acc[i][j][2 * h], acc[i][j][2 * h + 1]);
-                        } else {
-                            if (v0 + c < vdim) op[c] = acc[i][j][2 * h];
-                            if (v0 + c + 1 < vdim) op[c + 1] = acc[i][j][2 * h + 1];
-                        }
+                        if (v0 + c < vdim) *reinterpret_cast<float2*>(op + c) = make_float2(acc[i][j][2 * h], acc[i][j][2 * h + 1]);
                     }
                 }
         }
@@ -710,6 +720,9 @@ extern "C" int ns_delta_chunked(ns_device_t h, uint64_t q, int q_ld, uint64_t k,
     NS_REQUIRE(ns_source_ok(a_src, a_splits, NS_F32) && ns_source_ok(b_src, b_splits, NS_F32), NS_ERR_ARGUMENT, "ns_delta_chunked: bad source");
     NS_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0, NS_ERR_ARGUMENT, "ns_delta_chunked: %d heads do not divide over %d key heads", heads, kv_heads);
     NS_REQUIRE(dim > 0 && dim <= 128 && vdim > 0, NS_ERR_ARGUMENT, "ns_delta_chunked: key size %d (at most 128)", dim);
+    NS_REQUIRE(((dim | q_ld | k_ld) & 3) == 0 && ((q | k | dt_bias) & 15) == 0 && ((vdim | v_ld | o_ld) & 1) == 0 && ((v | o) & 7) == 0, NS_ERR_ARGUMENT,
+               "ns_delta_chunked: keys of %d and values of %d channels (multiples of 4 and 2, aligned)", dim, vdim);
+    NS_REQUIRE(!per_channel || (((a_ld | a_col) & 3) == 0 && (a_src & 15) == 0), NS_ERR_ARGUMENT, "ns_delta_chunked: decay projection not aligned");
     ChunkArgs a;
     const int64_t rows = (int64_t)batch * steps;
     a.q = reinterpret_cast<const float*>(q); a.q_ld = q_ld;

@@ -171,7 +171,7 @@ def run_delta(dev, data, cuts, H, kv, dim, vdim, channelwise, slots=(0,), chunk_
     for n in cuts:
         up = lambda z: dev.from_numpy(np.ascontiguousarray(z[:, at:at + n].reshape(B * n, -1), dtype=np.float32))
         dq, dk, dv = up(q), up(k), up(v)
-        ab, ld = split_source(dev, np.concatenate([a[:, at:at + n].reshape(B * n, ac), b[:, at:at + n].reshape(B * n, H)], 1), 2)
+        ab, ld = split_source(dev, np.concatenate([a[:, at:at + n].reshape(B * n, ac), b[:, at:at + n].reshape(B * n, H)], 1), 2, (ac + H + 7) // 8 * 8)
         o = dev.empty(B * n * H * vdim)
         N.call("ns_delta_chunked" if n >= chunk_from else "ns_delta_recurrent", dev.handle, u(dq.ptr), kv * dim, u(dk.ptr), kv * dim, u(dv.ptr), H * vdim, u(ab.ptr), 2, ld, 0, u(ab.ptr), 2, ld, ac,
                u(da.ptr), u(dd.ptr), int(channelwise), u(state.ptr), i64(stride), u(st.slots.ptr), B, n, H, kv, dim, vdim, u(o.ptr), H * vdim)
@@ -230,7 +230,7 @@ def test_delta_rule_over_cuts(dev, channelwise, cuts):
 
 @pytest.mark.parametrize("channelwise", [False, True])
 @pytest.mark.parametrize("T", [1, 16, 17, 63, 64, 65, 200])
-@pytest.mark.parametrize("H,kv,dim,vdim", [s for s in SIZES if s[2] <= 128] + [(2, 1, 33, 67)])
+@pytest.mark.parametrize("H,kv,dim,vdim", [s for s in SIZES if s[2] <= 128] + [(2, 1, 36, 66)])
 def test_delta_rule_in_chunks(dev, H, kv, dim, vdim, T, channelwise):
     data = delta_data(2, T, H, kv, dim, vdim, channelwise)
     o, s = run_delta(dev, data, (T,), H, kv, dim, vdim, channelwise, slots=(2, 0), chunk_from=1)
