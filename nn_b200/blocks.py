@@ -22,6 +22,10 @@ from .device import Device, _SIZE
 from .state import Reservation, SequenceStates
 
 
+# Passes of more rows than this (a prompt's portion) are bound by bytes, not by the number of launches.
+FEW_ROWS = 256
+
+
 def pad8(n: int) -> int:
     return (n + 7) // 8 * 8
 
@@ -97,9 +101,10 @@ def bf16_bits(a: np.ndarray) -> np.ndarray:
 
 class Product:
     """y = x . W^T for weights [n, k] given as bf16 bits (uint16) or float32; several matrices with the same input become one
-    product, their outputs side by side at ``cols``.  Input rows are ``k_ld`` long, output rows ``ld``."""
+    product, their outputs side by side at ``cols``.  Input rows are ``k_ld`` long, output rows ``ld``.  wide: the product is also
+    asked for as ``wide``."""
 
-    def __init__(self, ws: Workspace, *weights: np.ndarray):
+    def __init__(self, ws: Workspace, *weights: np.ndarray, wide: bool = False):
         self.dev, self.ws = ws.dev, ws
         k = weights[0].shape[1]
         self.cols, at = [], 0
@@ -118,6 +123,8 @@ class Product:
             ptr = C.c_uint64()
             N.call("ns_linear_info", h, None, None, None, C.byref(ptr), None, None)
             self.w_ptr = ptr.value
+            if wide:
+                ws.need("wide", self.ld)
         else:
             w = np.zeros((self.ld, self.k_ld), np.float32)
             w[:at, :k] = np.concatenate([f32(x) for x in weights])
@@ -135,6 +142,15 @@ class Product:
         N.call("ns_linear_forward_partial", self.dev.handle, self.handle, C.c_uint64(x), m, C.byref(ptr), C.byref(splits))
         step.launches += 1
         return Source(ptr.value, splits.value, N.NS_F32, self.ld)
+
+    def wide(self, x: int, step: Step) -> Source:
+        """The same for outputs that may be bf16: a pass of many rows (bf16 models) leaves one bf16 matrix in the workspace's "wide"
+        buffer, half the bytes of float sums; it stays until the next wide product."""
+        if self.handle is None or step.m <= FEW_ROWS:
+            return self(x, step)
+        self.into(x, step.m, self.ws["wide"], N.NS_BF16)
+        step.launches += 1
+        return Source(self.ws["wide"], 1, N.NS_BF16, self.ld)
 
     def into(self, x: int, m: int, y: int, dtype: int = N.NS_F32) -> None:
         """Output [m, ld] at y (bf16 layers: of either type)."""
@@ -167,12 +183,12 @@ class DenseGlu:
     def __init__(self, ws: Workspace, gate, up, down):
         self.dev, self.ws = ws.dev, ws
         self.ff = gate.shape[0]
-        self.gate_up = Product(ws, gate, up)
+        self.gate_up = Product(ws, gate, up, wide=True)
         self.down = Product(ws, down)
         ws.need("act", self.down.k_ld)
 
     def forward(self, h: int, step: Step) -> Source:
-        s = self.gate_up(h, step)
+        s = self.gate_up.wide(h, step)
         act = self.ws["act"]
         N.call("ns_glu_rows", self.dev.handle, *s.args, C.c_int64(step.m), self.ff, self.ws.dtype, C.c_uint64(act), self.down.k_ld)
         step.launches += 1
@@ -208,7 +224,8 @@ class DeltaMixer:
         self.channels = [kv_heads * dim, kv_heads * dim, heads * vdim]
         if self.channelwise:
             r1, r2 = w["a1"].shape[0], w["g1"].shape[0]
-            self.inputs = Product(ws, w["q"], w["k"], w["v"], w["b"], w["a1"], w["g1"])
+            names = ("b", "a1", "g1")
+            self.inputs = Product(ws, w["q"], w["k"], w["v"], *(w[n] for n in names), wide=True)
             # both low-rank pairs end in one product: block-diagonal, the outputs side by side
             second = np.zeros((heads * dim + heads * vdim, r1 + r2), np.float32)
             second[:heads * dim, :r1] = f32(w["a2"])
@@ -218,8 +235,11 @@ class DeltaMixer:
             ws.need("low_rank", self.second.k_ld)
             ws.need("beta", pad8(heads), N.NS_F32)
         else:
-            self.inputs = Product(ws, w["q"], w["k"], w["v"], w["b"], w["a"], w["g"])
+            names = ("b", "a")
+            self.inputs = Product(ws, w["q"], w["k"], w["v"], w["b"], w["a"], w["g"], wide=True)
             self.second = None
+        # what enters the recurrence besides q, k, v stays float where the rest of a long pass is bf16: its own small product
+        self.small = Product(ws, *(w[n] for n in names)) if ws.dtype == N.NS_BF16 else None
         self.out = Product(ws, w["o"])
         for n, c in zip("qkv", self.channels):
             ws.need("conv_" + n, c, N.NS_F32)
@@ -232,8 +252,8 @@ class DeltaMixer:
 
     def forward(self, h: int, cache: dict, step: Step) -> Source:
         ws, hd, H = self.ws, self.dev.handle, self.heads
-        s = self.inputs(h, step)
-        cols = self.inputs.cols
+        s = wide = self.inputs.wide(h, step)
+        cols = list(self.inputs.cols)
         fields, scales = [], []
         for i, n in enumerate("qkv"):
             heads, width = (H, self.vdim) if n == "v" else (self.kv_heads, self.dim)
@@ -242,13 +262,16 @@ class DeltaMixer:
         N.call("ns_short_conv", hd, *s.args, 3, (C.c_int64 * 27)(*fields), (C.c_float * 3)(*scales), C.c_int64(cache["hist"][0].stride),
                C.c_uint64(step.slots), C.c_uint64(step.pos), step.batch, step.steps, N.NS_F32)
         step.launches += 1
+        if wide.dtype == N.NS_BF16:
+            s = self.small(h, step)
+            cols[3:3 + len(self.small.cols)] = self.small.cols
         if self.channelwise:
             m = step.m
             N.call("ns_copy_cols", hd, *s.args, cols[3], C.c_int64(m), H, N.NS_F32, C.c_uint64(ws["beta"]), pad8(H))
             N.call("ns_copy_cols", hd, *s.args, cols[4], C.c_int64(m), self.low_rank, ws.dtype, C.c_uint64(ws["low_rank"]), self.second.k_ld)
             step.launches += 2
             beta, beta_col = Source(ws["beta"], 1, N.NS_F32, pad8(H)), 0
-            s = self.second(ws["low_rank"], step)
+            s = wide = self.second(ws["low_rank"], step)
             a_col, gate_col, act = 0, H * self.dim, N.ACT_SIGMOID
         else:
             beta, beta_col = s, cols[3]
@@ -258,13 +281,13 @@ class DeltaMixer:
         N.call("ns_delta_chunked" if self.chunks and step.steps >= self.CHUNK_STEPS else "ns_delta_recurrent", hd, u(ws["conv_q"]), self.channels[0], u(ws["conv_k"]), self.channels[1], u(ws["conv_v"]), self.channels[2],
                u(s.ptr), s.splits, s.ld, a_col, u(beta.ptr), beta.splits, beta.ld, beta_col, u(self.a_log.ptr), u(self.dt_bias.ptr), int(self.channelwise),
                u(state.ptr), C.c_int64(state.stride), u(step.slots), step.batch, step.steps, H, self.kv_heads, self.dim, self.vdim, u(ws["read"]), H * self.vdim)
-        N.call("ns_gated_norm", hd, u(ws["read"]), H * self.vdim, *s.args, gate_col, act, u(self.norm.ptr), C.c_float(self.eps), C.c_int64(step.m), H, self.vdim,
+        N.call("ns_gated_norm", hd, u(ws["read"]), H * self.vdim, *wide.args, gate_col, act, u(self.norm.ptr), C.c_float(self.eps), C.c_int64(step.m), H, self.vdim,
                ws.dtype, u(ws["mixed"]), self.out.k_ld)
         step.launches += 2
         return self.out(ws["mixed"], step)
 
     def close(self) -> None:
-        for p in (self.inputs, self.second, self.out):
+        for p in (self.inputs, self.second, self.small, self.out):
             if p is not None:
                 p.close()
 
@@ -291,7 +314,7 @@ class LatentAttentionMixer:
         i = np.arange(max(rot_dims // 2, 1), dtype=np.float64)
         self.freq = dev.from_numpy((float(rot_base) ** (-2.0 * i / max(rot_dims, 1))).astype(np.float32))
         self.down = Product(ws, w["dq"], w["dkv"])
-        self.uq = Product(ws, w["uq"])
+        self.uq = Product(ws, w["uq"], wide=True)
         # its input rows are whole cached rows: the columns of the rotated part are zero
         self.kv = Product(ws, *(np.pad(w[n], ((0, 0), (0, rot_dim))) for n in ("uk", "uv")))
         self.out = Product(ws, w["o"])
@@ -321,7 +344,7 @@ class LatentAttentionMixer:
         s = self.down(h, step)
         N.call("ns_latent_append", hd, *s.args, self.q_rank, R, self.rot_dim, self.rot_dims, u(self.q_norm.ptr), u(self.kv_norm.ptr), C.c_float(self.eps),
                u(self.freq.ptr), *at, dt, u(ws["cq"]), self.uq.k_ld, *ring_args)
-        s = self.uq(ws["cq"], step)
+        s = self.uq.wide(ws["cq"], step)
         rotate = (hd, *s.args, H, self.dim, self.rot_dim, self.rot_dims, u(self.freq.ptr), *at)
         mixed = ws[self.mixed]
         if self.expands and step.steps >= self.EXPAND_STEPS:

@@ -48,10 +48,19 @@ struct ConvArgs {
 // CTA share a head: 4 for prompts, 1 for the few tokens of a decoding step (the CTA then holds four heads).
 constexpr int CONV_WARP = 8;
 
-template <int V>
+enum { CONV_ANY = 0, CONV_F32 = 1, CONV_BF16 = 2 };   // what the source is: anything, one float matrix, one bf16 matrix
+
+template <int V, int SRC>
 NS_DEVINL void conv_load(const NsSource& s, int64_t idx, float (&x)[V])
 {
-    if constexpr (V == 4) {
+    if constexpr (SRC == CONV_F32 && V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(s.ptr) + idx);
+        x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+    } else if constexpr (SRC == CONV_BF16 && V == 4) {
+        const uint2 w = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(s.ptr) + idx);
+        x[0] = __uint_as_float(w.x << 16); x[1] = __uint_as_float(w.x & 0xFFFF0000u);
+        x[2] = __uint_as_float(w.y << 16); x[3] = __uint_as_float(w.y & 0xFFFF0000u);
+    } else if constexpr (V == 4) {
         const float4 t = ns_source_at4(s, idx);
         x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
     } else {
@@ -60,7 +69,7 @@ NS_DEVINL void conv_load(const NsSource& s, int64_t idx, float (&x)[V])
     }
 }
 
-template <typename T, int V, int TAPS>
+template <typename T, int V, int TAPS, int SRC = CONV_ANY>
 __global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs a, int span, int units)
 {
     ns_pdl_wait();
@@ -92,7 +101,7 @@ __global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs
             const int tt = t0 - n;
             if (n >= taps || pos0 + tt < 0) continue;
             if (tt >= 0) {
-                conv_load<V>(a.src, src0 + (int64_t)tt * a.src.ld, x[n - 1]);
+                conv_load<V, SRC>(a.src, src0 + (int64_t)tt * a.src.ld, x[n - 1]);
             } else {
                 const float* p = hist + (int64_t)((pos0 + tt) % taps) * channels;
 #pragma unroll
@@ -104,7 +113,7 @@ __global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs
     float in[CONV_WARP][V];
 #pragma unroll
     for (int j = 0; j < CONV_WARP; j++)
-        if (mine && t0 + j < t1) conv_load<V>(a.src, src0 + (int64_t)(t0 + j) * a.src.ld, in[j]);
+        if (mine && t0 + j < t1) conv_load<V, SRC>(a.src, src0 + (int64_t)(t0 + j) * a.src.ld, in[j]);
 #pragma unroll
     for (int j = 0; j < CONV_WARP; j++) {
         const int t = t0 + j;
@@ -142,7 +151,7 @@ __global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs
     if (blockIdx.x != 0 || (span == 4 && warp != 0) || !mine || taps < 2) return;
     for (int t = max(0, a.steps - (taps - 1)); t < a.steps; t++) {
         float v[V];
-        conv_load<V>(a.src, src0 + (int64_t)t * a.src.ld, v);
+        conv_load<V, SRC>(a.src, src0 + (int64_t)t * a.src.ld, v);
 #pragma unroll
         for (int i = 0; i < V; i++) hist[(int64_t)((pos0 + t) % taps) * channels + i] = v[i];
     }
@@ -500,6 +509,8 @@ extern "C" int ns_short_conv(ns_device_t h, uint64_t src, int splits, int src_dt
         };
         auto pick = [&](auto zero) -> int {
             using T = decltype(zero);
+            if (v == 4 && most_taps <= 4 && splits == 1 && steps > CONV_WARP)
+                return src_dtype == NS_F32 ? slide(ns_short_conv_slide_kernel<T, 4, 4, CONV_F32>) : slide(ns_short_conv_slide_kernel<T, 4, 4, CONV_BF16>);
             if (most_taps <= 4)
                 return v == 1 ? slide(ns_short_conv_slide_kernel<T, 1, 4>) : (v == 2 ? slide(ns_short_conv_slide_kernel<T, 2, 4>) : slide(ns_short_conv_slide_kernel<T, 4, 4>));
             return v == 1 ? slide(ns_short_conv_slide_kernel<T, 1, 8>) : (v == 2 ? slide(ns_short_conv_slide_kernel<T, 2, 8>) : slide(ns_short_conv_slide_kernel<T, 4, 8>));
