@@ -70,7 +70,7 @@ NS_DEVINL void conv_load(const NsSource& s, int64_t idx, float (&x)[V])
 }
 
 template <typename T, int V, int TAPS, int SRC = CONV_ANY>
-__global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs a, int span, int units)
+__global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs a, int span, int units, int pieces)
 {
     ns_pdl_wait();
     ns_pdl_trigger();
@@ -85,7 +85,8 @@ __global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs
     const bool mine = live && c < g.hd;
     float* hist = g.hist + (int64_t)slot * a.hist_slot_stride + ch;
     const int64_t src0 = (int64_t)b * a.steps * a.src.ld + g.col + ch;
-    const int t0 = span == 4 ? ((int)blockIdx.x * 4 + warp) * CONV_WARP : (int)blockIdx.x * CONV_WARP, t1 = min(t0 + CONV_WARP, a.steps);
+    const int per = CONV_WARP * pieces;
+    const int t0 = (span == 4 ? (int)blockIdx.x * 4 + warp : (int)blockIdx.x) * per, t1 = min(t0 + per, a.steps);
     float w[TAPS][V], x[TAPS][V];      // w[n]: weight of the input n tokens back; x[n]: that input
 #pragma unroll
     for (int n = 0; n < TAPS; n++)
@@ -109,39 +110,41 @@ __global__ void __launch_bounds__(128) ns_short_conv_slide_kernel(const ConvArgs
             }
         }
     }
-    // all inputs of the warp's tokens are on their way before the first is used
-    float in[CONV_WARP][V];
+    for (int tp = t0; tp < t1; tp += CONV_WARP) {
+        // all inputs of a piece are on their way before the first is used
+        float in[CONV_WARP][V];
 #pragma unroll
-    for (int j = 0; j < CONV_WARP; j++)
-        if (mine && t0 + j < t1) conv_load<V, SRC>(a.src, src0 + (int64_t)(t0 + j) * a.src.ld, in[j]);
+        for (int j = 0; j < CONV_WARP; j++)
+            if (mine && tp + j < t1) conv_load<V, SRC>(a.src, src0 + (int64_t)(tp + j) * a.src.ld, in[j]);
 #pragma unroll
-    for (int j = 0; j < CONV_WARP; j++) {
-        const int t = t0 + j;
-        if (t >= t1) break;
+        for (int j = 0; j < CONV_WARP; j++) {
+            const int t = tp + j;
+            if (t >= t1) break;
 #pragma unroll
-        for (int n = TAPS - 1; n > 0; n--)
+            for (int n = TAPS - 1; n > 0; n--)
 #pragma unroll
-            for (int i = 0; i < V; i++) x[n][i] = x[n - 1][i];
+                for (int i = 0; i < V; i++) x[n][i] = x[n - 1][i];
 #pragma unroll
-        for (int i = 0; i < V; i++) x[0][i] = mine ? in[j][i] : 0.0f;
-        float y[V], ss = 0.0f;
+            for (int i = 0; i < V; i++) x[0][i] = mine ? in[j][i] : 0.0f;
+            float y[V], ss = 0.0f;
 #pragma unroll
-        for (int i = 0; i < V; i++) {
-            float acc = 0.0f;
+            for (int i = 0; i < V; i++) {
+                float acc = 0.0f;
 #pragma unroll
-            for (int n = TAPS - 1; n >= 0; n--) acc = fmaf(x[n][i], w[n][i], acc);
-            y[i] = mine ? ns_silu(acc) : 0.0f;
-            ss = fmaf(y[i], y[i], ss);
-        }
-        float f = 1.0f;
-        if (g.unit) f = g.scale / sqrtf(ns_warp_sum(ss) + 1e-6f);
-        if (mine) {
-            T* out = reinterpret_cast<T*>(g.out) + ((int64_t)b * a.steps + t) * g.out_ld + ch;
-            if constexpr (V == 4) {
-                ns_store4(out, make_float4(y[0] * f, y[1] * f, y[2] * f, y[3] * f));
-            } else {
+                for (int n = TAPS - 1; n >= 0; n--) acc = fmaf(x[n][i], w[n][i], acc);
+                y[i] = mine ? __fdividef(acc, 1.0f + expf(-acc)) : 0.0f;
+                ss = fmaf(y[i], y[i], ss);
+            }
+            float f = 1.0f;
+            if (g.unit) f = g.scale / sqrtf(ns_warp_sum(ss) + 1e-6f);
+            if (mine) {
+                T* out = reinterpret_cast<T*>(g.out) + ((int64_t)b * a.steps + t) * g.out_ld + ch;
+                if constexpr (V == 4) {
+                    ns_store4(out, make_float4(y[0] * f, y[1] * f, y[2] * f, y[3] * f));
+                } else {
 #pragma unroll
-                for (int i = 0; i < V; i++) ns_store(out + i, y[i] * f);
+                    for (int i = 0; i < V; i++) ns_store(out + i, y[i] * f);
+                }
             }
         }
     }
@@ -501,10 +504,12 @@ extern "C" int ns_short_conv(ns_device_t h, uint64_t src, int splits, int src_dt
     if (v == 4 && ((src_ld & 3) != 0 || (src & 15) != 0)) v = 0;
     if (v != 0 && widest <= 128 && most_taps <= 8) {
         const int span = steps <= CONV_WARP ? 1 : 4;
-        const int per = span * CONV_WARP;
+        // a prompt's warps slide over four pieces: their weights and addresses are set up once
+        const int pieces = steps >= 256 ? 4 : 1;
+        const int per = span * CONV_WARP * pieces;
         const dim3 sgrid((unsigned)((steps + per - 1) / per), (unsigned)(span == 4 ? units : (units + 3) / 4), (unsigned)batch);
         auto slide = [&](auto k) -> int {
-            NS_CUDA(ns_launch_plain(k, sgrid, dim3(128), 0, d->stream, a, span, units));
+            NS_CUDA(ns_launch_plain(k, sgrid, dim3(128), 0, d->stream, a, span, units, pieces));
             return NS_OK;
         };
         auto pick = [&](auto zero) -> int {

@@ -80,12 +80,22 @@ NS_DEVINL void st_split4(uint32_t hi, uint32_t lo, float4 v)
     asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(lo), "r"(l0), "r"(l1) : "memory");
 }
 
-// log(1 + e^z) in 32-bit: the logarithm where 1 + e holds e's digits, its series below
+// log(1 + e^z) = max(z, 0) + log(1 + e), e = e^-|z| in (0, 1]; log(1 + e) / e by its Chebyshev interpolant of degree 9 on [0, 1]
+// (within 1.6e-7 of the value, evaluated in 32-bit), so that small e keep their digits and no lane branches.
 NS_DEVINL float softplus(float z)
 {
     const float e = ns_exp2(-fabsf(z) * LOG2E);
-    const float l = e < 0.015625f ? e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333333f), -0.5f), 1.0f) : logf(1.0f + e);
-    return fmaxf(z, 0.0f) + l;
+    float p = -0.00317605701f;
+    p = fmaf(p, e, 0.0195425283f);
+    p = fmaf(p, e, -0.0563736148f);
+    p = fmaf(p, e, 0.105436236f);
+    p = fmaf(p, e, -0.152696669f);
+    p = fmaf(p, e, 0.196632743f);
+    p = fmaf(p, e, -0.249516159f);
+    p = fmaf(p, e, 0.333297104f);
+    p = fmaf(p, e, -0.499998927f);
+    p = fmaf(p, e, 1.0f);
+    return fmaf(e, p, fmaxf(z, 0.0f));
 }
 
 template <int DK, int DV>
