@@ -9,12 +9,19 @@
 //
 // Scores, maxima, sums and accumulators are 32-bit; the operands of the two products (queries, keys, values, softmax weights) are
 // bf16 as in the full-attention kernels.
+#include <string.h>
+
 #include "ns_mma.cuh"
 #include "ns_seq.cuh"
 
 namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
+
+NS_DEVINL void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar)
+{
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
 
 // ---------------------------------------------------------------------------------------------
 // gather
@@ -48,19 +55,40 @@ struct PrefillArgs {
     int steps, heads, dim, rot, vdim, past, nk, window;
     float scale2;                            // scale * log2(e)
     int vec;
+    int dim_boxes;                           // TMA: boxes of the unrotated part
+    int* status;
+};
+struct PrefillMaps {
+    CUtensorMap kv, keys;                    // boxes of 64 columns x 64 rows
 };
 
 constexpr int PF_ROWS = 64, PF_KEYS = 64;
+constexpr uint32_t PF_BOX = 64 * 128;       // bytes
 
 // NV: value n-tiles of 8.  KS: 16-wide k-steps of the scores whose query fragments stay in registers.
-template <int NV, int KS>
-__global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArgs a)
+// TMA: key and value tiles arrive as boxes of 64 columns x 64 rows (128-byte swizzle), the unrotated and the rotated part of the
+// heads each padded to whole boxes.  What a box holds beyond its part meets zeros of the query, or columns that are not stored.
+// Otherwise (sizes that are not multiples of 8) rows are copied piece by piece.
+template <int NV, int KS, bool TMA>
+__global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const __grid_constant__ PrefillMaps maps, const PrefillArgs a)
 {
-    extern __shared__ __align__(16) uint16_t pf_smem[];
+    extern __shared__ __align__(1024) uint16_t pf_smem[];
     constexpr int VLD = NV * 8 + 8, DKP = KS * 16, KLD = DKP + 8;
+    constexpr int KB = KS / 4, VB = (NV + 7) / 8;        // boxes of a key and of a value tile
+    constexpr uint32_t K_BYTES = TMA ? KB * PF_BOX : PF_KEYS * KLD * 2, V_BYTES = TMA ? VB * PF_BOX : PF_KEYS * VLD * 2;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-    const uint32_t sK = ns_smem_u32(pf_smem), sV = sK + 2 * PF_KEYS * KLD * 2;
-    const uint32_t sQ = sK + PF_KEYS * KLD * 2;          // the second key stage, before it is filled
+    const uint32_t raw = ns_smem_u32(pf_smem), sK = TMA ? (raw + 1023u) & ~1023u : raw, sV = sK + 2 * K_BYTES;
+    const uint32_t sQ = TMA ? sV : sK + K_BYTES;         // a place that is filled after the query fragments have been read
+    __shared__ __align__(8) uint64_t full[2];
+    __shared__ int abort_flag;
+    const uint32_t bars = ns_smem_u32(full);
+    if (TMA && tid == 0) {
+        abort_flag = 0;
+        ns_mbar_init(bars, 1);
+        ns_mbar_init(bars + 8, 1);
+        ns_fence_barrier_init();
+        ns_fence_proxy_async();
+    }
     ns_pdl_wait();
     ns_pdl_trigger();
     const int tiles_q = (a.steps + PF_ROWS - 1) / PF_ROWS;
@@ -72,10 +100,31 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
     for (int r = warp; r < PF_ROWS; r += 4) {
         const bool in = q0 + r < a.steps;
         const uint16_t* src = a.q + ((int64_t)b * a.steps + (in ? q0 + r : 0)) * a.q_ld + (int64_t)head * dk;
-        for (int c = lane * 8; c < DKP; c += 256) ns_copy8(sQ + (r * KLD + c) * 2, src + (in && c < dk ? c : 0), in ? dk - c : 0, a.vec);
+        for (int c = lane * 8; c < DKP; c += 256) {
+            int at = c, left = dk - c;                   // column of the head and how many follow it in its part
+            if (TMA) {
+                const bool plain = c < a.dim_boxes * 64;
+                at = plain ? c : a.dim + c - a.dim_boxes * 64;
+                left = plain ? a.dim - c : dk - at;
+            }
+            ns_copy8(sQ + (r * KLD + c) * 2, src + (in && left > 0 ? at : 0), in ? left : 0, a.vec);
+        }
     }
     auto load_tile = [&](int kt, int stage) {
         const int k0 = kt * PF_KEYS;
+        if (TMA) {
+            if (tid == 0) {
+                const uint32_t bar = bars + 8 * stage, dk_s = sK + stage * K_BYTES, dv_s = sV + stage * V_BYTES;
+                const int y = b * a.nk + k0;
+                ns_mbar_expect_tx(bar, K_BYTES + V_BYTES);
+                for (int i = 0; i < KB; i++) {
+                    if (i < a.dim_boxes) ns_tma_load_2d(dk_s + i * PF_BOX, &maps.kv, bar, head * a.dim + i * 64, y);
+                    else ns_tma_load_2d(dk_s + i * PF_BOX, &maps.keys, bar, a.rank + (i - a.dim_boxes) * 64, y);
+                }
+                for (int i = 0; i < VB; i++) ns_tma_load_2d(dv_s + i * PF_BOX, &maps.kv, bar, a.heads * a.dim + head * a.vdim + i * 64, y);
+            }
+            return;
+        }
         const uint32_t dk_s = sK + stage * PF_KEYS * KLD * 2, dv_s = sV + stage * PF_KEYS * VLD * 2;
         for (int r = warp; r < PF_KEYS; r += 4) {
             const bool in = k0 + r < a.nk;
@@ -127,23 +176,43 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
     const int r0 = q0 + warp * 16 + g;       // query rows r0 and r0 + 8
 
-    load_tile(t_first, 0);
+    if (TMA) ns_cp_commit();
+    else load_tile(t_first, 0);
     ns_cp_wait<0>();
     __syncthreads();
     uint32_t qf[KS][4];
 #pragma unroll
     for (int k = 0; k < KS; k++) ns_ldsm4(qf[k], ns_addr_a(sQ, KLD, warp * 16, k * 16, lane));
     __syncthreads();
+    if (TMA) {
+        ns_fence_proxy_async();          // the query's place was written and read by the generic proxy
+        load_tile(t_first, 0);
+    }
+    bool gave_up = false;
     for (int kt = t_first; kt <= t_last; kt++) {
         const int stage = (kt - t_first) & 1;
-        if (kt < t_last) {
-            load_tile(kt + 1, stage ^ 1);
-            ns_cp_wait<1>();
+        if (kt < t_last) load_tile(kt + 1, stage ^ 1);
+        if (TMA) {
+            const bool ok = ns_mbar_wait(bars + 8 * stage, ((kt - t_first) >> 1) & 1, &abort_flag, a.status, 710);
+            if (__syncthreads_or(!ok)) {
+                gave_up = true;
+                break;
+            }
         } else {
-            ns_cp_wait<0>();
+            if (kt < t_last) ns_cp_wait<1>();
+            else ns_cp_wait<0>();
+            __syncthreads();
         }
-        __syncthreads();
-        const uint32_t tK = sK + stage * PF_KEYS * KLD * 2, tV = sV + stage * PF_KEYS * VLD * 2;
+        const uint32_t tK = sK + stage * K_BYTES, tV = sV + stage * V_BYTES;
+        // ldmatrix addresses of 16 keys x 16 columns, and of 16 keys x 16 value columns (transposed)
+        auto key_addr = [&](int n, int k) -> uint32_t {
+            if (TMA) return tK + (k >> 6) * PF_BOX + (n + (lane & 7) + (lane >> 4) * 8) * 128 + (((((k & 63) >> 3) + ((lane >> 3) & 1)) ^ (lane & 7)) * 16);
+            return ns_addr_b(tK, KLD, n, k, lane);
+        };
+        auto value_addr = [&](int k, int n) -> uint32_t {
+            if (TMA) return tV + (n >> 6) * PF_BOX + (k + (lane & 7) + ((lane >> 3) & 1) * 8) * 128 + (((((n & 63) >> 3) + (lane >> 4)) ^ (lane & 7)) * 16);
+            return ns_addr_bt(tV, VLD, k, n, lane);
+        };
         float s[8][4];
 #pragma unroll
         for (int j = 0; j < 8; j++)
@@ -152,12 +221,12 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
         // the next k-step's key fragments are on their way while this one is multiplied
         uint32_t bf[2][4][4];
 #pragma unroll
-        for (int j = 0; j < 4; j++) ns_ldsm4(bf[0][j], ns_addr_b(tK, KLD, j * 16, 0, lane));
+        for (int j = 0; j < 4; j++) ns_ldsm4(bf[0][j], key_addr(j * 16, 0));
 #pragma unroll
         for (int k = 0; k < KS; k++) {
             if (k + 1 < KS)
 #pragma unroll
-                for (int j = 0; j < 4; j++) ns_ldsm4(bf[(k + 1) & 1][j], ns_addr_b(tK, KLD, j * 16, (k + 1) * 16, lane));
+                for (int j = 0; j < 4; j++) ns_ldsm4(bf[(k + 1) & 1][j], key_addr(j * 16, (k + 1) * 16));
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 ns_mma_bf16(s[2 * j], qf[k], bf[k & 1][j][0], bf[k & 1][j][1]);
@@ -208,7 +277,7 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
         constexpr int GV = NV >= 8 ? 4 : NV / 2, NG = NV / 2 / GV;      // value fragments in groups of GV, one group ahead
         uint32_t vf[2][GV][4];
 #pragma unroll
-        for (int j = 0; j < GV; j++) ns_ldsm4_t(vf[0][j], ns_addr_bt(tV, VLD, 0, j * 16, lane));
+        for (int j = 0; j < GV; j++) ns_ldsm4_t(vf[0][j], value_addr(0, j * 16));
 #pragma unroll
         for (int k = 0; k < 4; k++) {
             const uint32_t pf[4] = {ns_pack_bf16x2(s[2 * k][0], s[2 * k][1]), ns_pack_bf16x2(s[2 * k][2], s[2 * k][3]),
@@ -218,7 +287,7 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
                 const int at = k * NG + q, nx = at + 1;
                 if (nx < 4 * NG)
 #pragma unroll
-                    for (int j = 0; j < GV; j++) ns_ldsm4_t(vf[nx & 1][j], ns_addr_bt(tV, VLD, (nx / NG) * 16, ((nx % NG) * GV + j) * 16, lane));
+                    for (int j = 0; j < GV; j++) ns_ldsm4_t(vf[nx & 1][j], value_addr((nx / NG) * 16, ((nx % NG) * GV + j) * 16));
 #pragma unroll
                 for (int j = 0; j < GV; j++) {
                     ns_mma_bf16(acc[2 * (q * GV + j)], pf, vf[at & 1][j][0], vf[at & 1][j][1]);
@@ -227,6 +296,11 @@ __global__ void __launch_bounds__(128) ns_latent_prefill_kernel(const PrefillArg
             }
         }
         __syncthreads();
+    }
+    if (gave_up) {                       // copies of this CTA may still be in flight: leave them time to land
+        const long long t0 = clock64();
+        while (clock64() - t0 < 400000) { }
+        return;
     }
 #pragma unroll
     for (int h = 0; h < 2; h++) {
@@ -268,6 +342,7 @@ struct DecodeArgs {
     uint16_t* o;               // [batch, rows, rank]; splits == 1
     float* part;               // [batch, rows, splits, rank + 2]: weighted sum, maximum, sum
     int splits;
+    int* status;
 };
 
 constexpr int DC_KEYS = 64;
@@ -282,6 +357,16 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
     const uint32_t sQ = ns_smem_u32(dc_smem), sC = sQ + R * ld * 2, sP = sC + 2 * DC_KEYS * ld * 2;
     float* sS = reinterpret_cast<float*>(dc_smem + (size_t)(R + 2 * DC_KEYS) * ld + R * PLD);
     float* sF = sS + R * SLD;                 // rescale factor of a row, then its 1 / sum
+    __shared__ __align__(8) uint64_t full[2];
+    __shared__ int abort_flag;
+    const uint32_t bars = ns_smem_u32(full);
+    if (tid == 0) {
+        abort_flag = 0;
+        ns_mbar_init(bars, 1);
+        ns_mbar_init(bars + 8, 1);
+        ns_fence_barrier_init();
+        ns_fence_proxy_async();
+    }
     ns_pdl_wait();
     ns_pdl_trigger();
     const int b = blockIdx.z, row0 = blockIdx.y * R, split = blockIdx.x;
@@ -296,17 +381,25 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
         const uint16_t* src = a.q + ((int64_t)b * a.rows + (in ? row0 + r : 0)) * a.width;
         for (int c = lane * 8; c < a.wp; c += 256) ns_copy8(sQ + (r * ld + c) * 2, src + (c < a.width ? c : 0), in ? a.width - c : 0, (a.width & 7) == 0);
     }
-    // a warp per cached row; rows are padded to a multiple of 8 with zeros
+    // columns past the cached row stay zero
+    for (int r = warp; r < 2 * DC_KEYS; r += 8)
+        for (int c = a.ring_ld + lane * 8; c < a.wp; c += 256) ns_st_shared_v4(sC + (r * ld + c) * 2, 0, 0, 0, 0);
+    ns_cp_commit();
+    ns_cp_wait<0>();
+    __syncthreads();
+    // Warp 0 orders the rows of a tile as one bulk copy each; rows past the last position become zero.
     auto load_tile = [&](int t, int stage) {
-        const int p0 = first + t * DC_KEYS;
-#pragma unroll 2
-        for (int r = warp; r < DC_KEYS; r += 8) {
-            const bool in = p0 + r <= last;
-            const uint16_t* src = ring + (int64_t)(in ? (p0 + r) % a.ring_len : 0) * a.ring_ld;
-            for (int c = lane * 8; c < a.wp; c += 256)
-                ns_copy8(sC + ((stage * DC_KEYS + r) * ld + c) * 2, src + (c < a.ring_ld ? c : 0), in ? a.ring_ld - c : 0, true);
+        const int p0 = first + t * DC_KEYS, count = min(DC_KEYS, last - p0 + 1);
+        if (warp == 0) {
+            const uint32_t bar = bars + 8 * stage, bytes = a.ring_ld * 2;
+            if (lane == 0) ns_mbar_expect_tx(bar, count * bytes);
+            __syncwarp();
+            for (int r = lane; r < count; r += 32)
+                bulk_load(sC + (stage * DC_KEYS + r) * ld * 2, ring + (int64_t)((p0 + r) % a.ring_len) * a.ring_ld, bytes, bar);
+        } else if (count < DC_KEYS) {
+            for (int r = count + warp - 1; r < DC_KEYS; r += 7)
+                for (int c = lane * 8; c < a.ring_ld; c += 256) ns_st_shared_v4(sC + ((stage * DC_KEYS + r) * ld + c) * 2, 0, 0, 0, 0);
         }
-        ns_cp_commit();
     };
 
     float acc[MT][NW][4];
@@ -324,13 +417,9 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
     if (tb < te) load_tile(tb, 0);
     for (int t = tb; t < te; t++) {
         const int stage = (t - tb) & 1;
-        if (t + 1 < te) {
-            load_tile(t + 1, stage ^ 1);
-            ns_cp_wait<1>();
-        } else {
-            ns_cp_wait<0>();
-        }
-        __syncthreads();
+        if (t + 1 < te) load_tile(t + 1, stage ^ 1);
+        const bool ok = ns_mbar_wait(bars + 8 * stage, ((t - tb) >> 1) & 1, &abort_flag, a.status, 700);
+        if (__syncthreads_or(!ok)) break;
         const uint32_t tC = sC + stage * DC_KEYS * ld * 2;
         // scores: warp w takes keys 8w .. 8w + 7
         // two chains of accumulation per row tile
@@ -409,6 +498,10 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
         __syncthreads();
     }
 
+    if (abort_flag != 0) {                    // copies of this CTA may still be in flight: leave them time to land
+        const long long t0 = clock64();
+        while (clock64() - t0 < 400000) { }
+    }
     if (a.splits == 1) {
 #pragma unroll
         for (int i = 0; i < 2 * MT; i++)
@@ -535,25 +628,33 @@ __global__ void __launch_bounds__(128) ns_head_matmul_tc_kernel(const HeadTcArgs
         }
 }
 
-template <int NV, int KS>
-int launch_prefill(NsDevice* d, const PrefillArgs& a, int batch)
+template <int NV, int KS, bool TMA>
+int launch_prefill(NsDevice* d, const PrefillMaps& maps, const PrefillArgs& a, int batch)
 {
-    constexpr size_t smem = ((size_t)2 * PF_KEYS * (KS * 16 + 8) + 2 * PF_KEYS * (NV * 8 + 8)) * 2;
+    constexpr size_t rows = ((size_t)2 * PF_KEYS * (KS * 16 + 8) + 2 * PF_KEYS * (NV * 8 + 8)) * 2;
+    constexpr size_t boxes = 1024 + 2 * ((size_t)KS / 4 + (NV + 7) / 8) * PF_BOX, q_end = 1024 + 2 * (size_t)(KS / 4) * PF_BOX + PF_ROWS * (KS * 16 + 8) * 2;
+    constexpr size_t smem = TMA ? (boxes > q_end ? boxes : q_end) : rows;
     static_assert(smem <= 227 * 1024, "tiles do not fit shared memory");
-    auto k = ns_latent_prefill_kernel<NV, KS>;
+    auto k = ns_latent_prefill_kernel<NV, KS, TMA>;
     NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    NS_CUDA(ns_launch_plain(k, dim3((a.steps + PF_ROWS - 1) / PF_ROWS, a.heads, batch), dim3(128), smem, d->stream, a));
+    NS_CUDA(ns_launch_plain(k, dim3((a.steps + PF_ROWS - 1) / PF_ROWS, a.heads, batch), dim3(128), smem, d->stream, maps, a));
     return NS_OK;
 }
 
 template <int NV>
-int dispatch_prefill(NsDevice* d, const PrefillArgs& a, int batch)
+int dispatch_prefill(NsDevice* d, const PrefillMaps& maps, const PrefillArgs& a, int batch, int boxes)
 {
-    const int dk = a.dim + a.rot;
-    if (dk <= 64) return launch_prefill<NV, 4>(d, a, batch);
-    if (dk <= 128) return launch_prefill<NV, 8>(d, a, batch);
-    if (dk <= 192) return launch_prefill<NV, 12>(d, a, batch);
-    return launch_prefill<NV, 16>(d, a, batch);
+    if (boxes == 0) {
+        const int dk = a.dim + a.rot;
+        if (dk <= 64) return launch_prefill<NV, 4, false>(d, maps, a, batch);
+        if (dk <= 128) return launch_prefill<NV, 8, false>(d, maps, a, batch);
+        if (dk <= 192) return launch_prefill<NV, 12, false>(d, maps, a, batch);
+        return launch_prefill<NV, 16, false>(d, maps, a, batch);
+    }
+    if (boxes == 1) return launch_prefill<NV, 4, true>(d, maps, a, batch);
+    if (boxes == 2) return launch_prefill<NV, 8, true>(d, maps, a, batch);
+    if (boxes == 3) return launch_prefill<NV, 12, true>(d, maps, a, batch);
+    return launch_prefill<NV, 16, true>(d, maps, a, batch);
 }
 
 template <int MT, int NW>
@@ -607,10 +708,26 @@ extern "C" int ns_latent_prefill(ns_device_t h, uint64_t q, int64_t q_ld, uint64
     a.steps = steps; a.heads = heads; a.dim = dim; a.rot = rot_dim; a.vdim = vdim; a.past = past; a.nk = past + steps; a.window = window;
     a.scale2 = scale * LOG2E;
     a.vec = ((dim | rot_dim | vdim | rank | (int)q_ld | (int)kv_ld | (int)keys_ld) & 7) == 0 && ((q | kv | keys) & 15) == 0;
-    if (vdim <= 32) return dispatch_prefill<4>(d, a, batch);
-    if (vdim <= 64) return dispatch_prefill<8>(d, a, batch);
-    if (vdim <= 128) return dispatch_prefill<16>(d, a, batch);
-    return dispatch_prefill<32>(d, a, batch);
+    a.status = d->status_dev;
+    a.dim_boxes = (dim + 63) / 64;
+    const int boxes = a.dim_boxes + (rot_dim + 63) / 64;
+    const bool tma = a.vec && boxes <= 4 && (int64_t)batch * a.nk < (1ll << 31);
+    PrefillMaps maps;
+    memset(&maps, 0, sizeof(maps));
+    if (tma) {
+        const uint64_t rows = (uint64_t)batch * a.nk;
+        const uint32_t box[2] = {64, 64};
+        const uint64_t kv_dims[2] = {(uint64_t)kv_ld, rows}, kv_strides[1] = {(uint64_t)kv_ld * 2};
+        const uint64_t key_dims[2] = {(uint64_t)keys_ld, rows}, key_strides[1] = {(uint64_t)keys_ld * 2};
+        int rc = ns_make_tensor_map(&maps.kv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kv, kv_dims, kv_strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
+        if (rc == NS_OK) rc = ns_make_tensor_map(&maps.keys, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.keys, key_dims, key_strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
+        if (rc != NS_OK) return rc;
+    }
+    const int n = tma ? boxes : 0;
+    if (vdim <= 32) return dispatch_prefill<4>(d, maps, a, batch, n);
+    if (vdim <= 64) return dispatch_prefill<8>(d, maps, a, batch, n);
+    if (vdim <= 128) return dispatch_prefill<16>(d, maps, a, batch, n);
+    return dispatch_prefill<32>(d, maps, a, batch, n);
 }
 
 extern "C" int ns_latent_decode(ns_device_t h, uint64_t q, uint64_t ring, int64_t ring_slot_stride, int ring_len, int ring_ld, int rank, int width, int window,
@@ -628,6 +745,7 @@ extern "C" int ns_latent_decode(ns_device_t h, uint64_t q, uint64_t ring, int64_
     a.slots = I32P(slots); a.pos = I32P(pos); a.steps = steps; a.heads = heads; a.rows = steps * heads;
     a.o = reinterpret_cast<uint16_t*>(o);
     a.part = nullptr;
+    a.status = d->status_dev;
     const bool two = a.rows > 16 && rank <= 512;
     const int R = two ? 32 : 16;
     const int64_t ctas = (int64_t)batch * ((a.rows + R - 1) / R);
