@@ -4,7 +4,7 @@
 //   ns_latent_prefill  a prompt's portion: keys and values already expanded per head, windowed causal attention over 64-row
 //                      query tiles and 64-key tiles, one warp per 16 query rows
 //   ns_latent_decode   few tokens: attention over the cached latents themselves; all heads of a sequence share the cached rows,
-//                      so a tile of 64 rows is read once for 16 or 32 (token, head) rows
+//                      so a tile of 32 rows is read once for 16 or 32 (token, head) rows
 //   ns_head_matmul_tc  the per-head products around it
 //
 // Scores, maxima, sums and accumulators are 32-bit; the operands of the two products (queries, keys, values, softmax weights) are
@@ -345,18 +345,18 @@ struct DecodeArgs {
     int* status;
 };
 
-constexpr int DC_KEYS = 64;
+constexpr int DC_KEYS = 32;
 
 // MT: 16-row tiles per CTA; NW: value n-tiles of 8 per warp (8 warps side by side over the latent)
 template <int MT, int NW>
-__global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs a)
+__global__ void __launch_bounds__(256, MT == 1 && NW <= 8 ? 2 : 1) ns_latent_decode_kernel(const DecodeArgs a)
 {
     extern __shared__ __align__(16) uint16_t dc_smem[];
     constexpr int R = MT * 16, SLD = DC_KEYS + 4, PLD = DC_KEYS + 8;
     const int ld = a.wp + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const uint32_t sQ = ns_smem_u32(dc_smem), sC = sQ + R * ld * 2, sP = sC + 2 * DC_KEYS * ld * 2;
     float* sS = reinterpret_cast<float*>(dc_smem + (size_t)(R + 2 * DC_KEYS) * ld + R * PLD);
-    float* sF = sS + R * SLD;                 // rescale factor of a row, then its 1 / sum
+    float* sF = sS + 2 * R * SLD;             // rescale factor of a row, then its 1 / sum
     __shared__ __align__(8) uint64_t full[2];
     __shared__ int abort_flag;
     const uint32_t bars = ns_smem_u32(full);
@@ -421,17 +421,17 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
         const bool ok = ns_mbar_wait(bars + 8 * stage, ((t - tb) >> 1) & 1, &abort_flag, a.status, 700);
         if (__syncthreads_or(!ok)) break;
         const uint32_t tC = sC + stage * DC_KEYS * ld * 2;
-        // scores: warp w takes keys 8w .. 8w + 7
-        // two chains of accumulation per row tile
+        // scores: four warps share the keys, 8 each, for the first half of the columns, four for the second
+        const int kq = (warp & 3) * 8, half = warp >> 2, k_mid = (a.wp / 32 + 1) / 2 * 32;
         float s[MT][4], s2[MT][4];
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
             for (int k = 0; k < 4; k++) s[i][k] = s2[i][k] = 0.0f;
 #pragma unroll 4
-        for (int k = 0; k < a.wp; k += 32) {
+        for (int k = half ? k_mid : 0; k < (half ? a.wp : k_mid); k += 32) {
             uint32_t bf[4];
-            ns_ldsm4(bf, tC + ((warp * 8 + (lane & 7)) * ld + k + (lane >> 3) * 8) * 2);
+            ns_ldsm4(bf, tC + ((kq + (lane & 7)) * ld + k + (lane >> 3) * 8) * 2);
 #pragma unroll
             for (int i = 0; i < MT; i++) {
                 uint32_t af[4], ag[4];
@@ -444,30 +444,22 @@ __global__ void __launch_bounds__(256) ns_latent_decode_kernel(const DecodeArgs 
 #pragma unroll
         for (int i = 0; i < MT; i++)
 #pragma unroll
-            for (int k = 0; k < 4; k++) s[i][k] += s2[i][k];
-        const int p0 = first + t * DC_KEYS;
-#pragma unroll
-        for (int i = 0; i < MT; i++)
-#pragma unroll
-            for (int k = 0; k < 4; k++) {
-                const int r = i * 16 + g + (k >> 1) * 8, c = warp * 8 + t4 * 2 + (k & 1);
-                const int at = pos0 + (row0 + r) / a.heads, key = p0 + c;
-                const bool see = key <= at && (a.window <= 0 || key > at - a.window);
-                sS[r * SLD + c] = see ? s[i][k] * a.scale2 : -INFINITY;
-            }
+            for (int k = 0; k < 4; k++) sS[(half * R + i * 16 + g + (k >> 1) * 8) * SLD + kq + t4 * 2 + (k & 1)] = s[i][k] + s2[i][k];
         __syncthreads();
+        const int key = first + t * DC_KEYS + lane;
 #pragma unroll
         for (int i = 0; i < 2 * MT; i++) {
-            const int r = warp * 2 * MT + i;
-            const float s0 = sS[r * SLD + 2 * lane], s1 = sS[r * SLD + 2 * lane + 1];
-            float mt = fmaxf(s0, s1);
+            const int r = warp * 2 * MT + i, at = pos0 + (row0 + r) / a.heads;
+            const bool see = key <= at && (a.window <= 0 || key > at - a.window);
+            const float s0 = see ? (sS[r * SLD + lane] + sS[(R + r) * SLD + lane]) * a.scale2 : -INFINITY;
+            float mt = s0;
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, o));
             const float mn = fmaxf(m[i], mt), base = mn == -INFINITY ? 0.0f : mn;
-            const float f = ns_exp2(m[i] - base), e0 = ns_exp2(s0 - base), e1 = ns_exp2(s1 - base);
-            l[i] = fmaf(l[i], f, ns_warp_sum(e0 + e1));
+            const float f = ns_exp2(m[i] - base), e0 = ns_exp2(s0 - base);
+            l[i] = fmaf(l[i], f, ns_warp_sum(e0));
             m[i] = mn;
-            asm volatile("st.shared.b32 [%0], %1;" ::"r"(sP + (r * PLD + 2 * lane) * 2), "r"(ns_pack_bf16x2(e0, e1)) : "memory");
+            asm volatile("st.shared.b16 [%0], %1;" ::"r"(sP + (r * PLD + lane) * 2), "h"(ns_f32_to_bf16_bits(e0)) : "memory");
             if (lane == 0) sF[r] = f;
         }
         __syncthreads();
@@ -661,7 +653,7 @@ template <int MT, int NW>
 int launch_decode(NsDevice* d, const DecodeArgs& a, int batch)
 {
     constexpr int R = MT * 16;
-    const size_t smem = ((size_t)(R + 2 * DC_KEYS) * (a.wp + 8) + R * (DC_KEYS + 8)) * 2 + (size_t)(R * (DC_KEYS + 4) + R) * 4;
+    const size_t smem = ((size_t)(R + 2 * DC_KEYS) * (a.wp + 8) + R * (DC_KEYS + 8)) * 2 + (size_t)(2 * R * (DC_KEYS + 4) + R) * 4;
     NS_REQUIRE(smem <= 227 * 1024, NS_ERR_ARGUMENT, "ns_latent_decode: cached rows of %d values do not fit shared memory", a.width);
     auto k = ns_latent_decode_kernel<MT, NW>;
     NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -750,9 +742,9 @@ extern "C" int ns_latent_decode(ns_device_t h, uint64_t q, uint64_t ring, int64_
     const int R = two ? 32 : 16;
     const int64_t ctas = (int64_t)batch * ((a.rows + R - 1) / R);
     NS_REQUIRE((a.rows + R - 1) / R <= 65535, NS_ERR_ARGUMENT, "ns_latent_decode: too many rows");
-    // about one CTA per SM (the two tiles in flight fill its shared memory), at least two tiles of keys each
+    // about two CTAs per SM, at least two tiles of keys each
     const int span = window > 0 ? window - 1 + steps : ring_len;
-    int splits = (int)(d->sm_count / ctas);
+    int splits = (int)(2 * d->sm_count / ctas);
     const int most = (span / DC_KEYS + 1) / 2;
     if (splits > most) splits = most;
     if (splits > 16) splits = 16;
