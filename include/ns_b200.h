@@ -418,8 +418,8 @@ NS_API int ns_linear_forward_kv_append(ns_device_t dev, ns_linear_t linear, uint
  * states are given as slot 0's address and the stride between slots in elements.  Rows are [batch, steps].
  * Outputs that feed a product are written with a row pitch `*_ld` >= their width, padded with zeros.
  * ------------------------------------------------------------------------------------------------ */
-/* y[b, i, :] = scale * table[token] + bigram[row], row = (previous token * mul_prev + token * mul_cur) mod buckets, and row
- * `buckets` (the table's last) for a sequence's first token.  bigram may be 0.  Tables [rows, ld] of table_dtype, y float. */
+/* y[b, i, :] = scale * table[token] + bigram[row], row = (p * mul_prev + t * mul_cur) mod buckets for token t after
+ * token p, and `buckets` (one past the hashed rows) where nothing comes before t.  bigram may be 0.  Tables [rows, ld] of table_dtype, y float. */
 NS_API int ns_embed_ngram(ns_device_t dev, uint64_t ids, uint64_t table, int table_dtype, int table_ld, float scale, uint64_t bigram, int bigram_ld,
                           int buckets, int64_t mul_prev, int64_t mul_cur, uint64_t slots, uint64_t last, int batch, int steps, int dim, int vocab, uint64_t y);
 /* x_out = x + alpha * source (float; x or the source may be 0; x_out may be 0 or x), then, when w != 0,
@@ -437,8 +437,8 @@ NS_API int ns_seq_advance(ns_device_t dev, uint64_t ids, uint64_t slots, int bat
 /* int32 ids from the float-encoded ones of the sampler (ns_f32_sample_rows) */
 NS_API int ns_ids_from_f32(ns_device_t dev, uint64_t x, uint64_t ids, int n);
 
-/* Causal convolution over time per channel, then silu, then optionally every head made a unit vector
- * (x / sqrt(sum x^2 + 1e-6)) times scales[s], for up to 4 tensors that lie side by side in the source.  fields: 9 int64 per
+/* Causal convolution over time per channel, then silu, then optionally every head scaled to length
+ * scales[s] (1e-6 added to its squared length), for up to 4 tensors that lie side by side in the source.  fields: 9 int64 per
  * tensor: first column, heads, channels per head, taps, unit (0 / 1), weight address (float [channels, taps], the current
  * token's last), history address of slot 0 (float [taps, channels]: the raw inputs of earlier tokens at position modulo taps),
  * output address ([rows, ld] of out_dtype), output ld.  The history of the step's sequences is read and replaced. */
@@ -446,7 +446,7 @@ NS_API int ns_short_conv(ns_device_t dev, uint64_t src, int splits, int src_dtyp
                          int64_t hist_slot_stride, uint64_t slots, uint64_t pos, int batch, int steps, int out_dtype);
 /* Gated delta rule, token by token, in 32-bit floats: per head a state S [dim, vdim];
  *   g = exp(-exp(a_log) * softplus(a + dt_bias)), beta = sigmoid(b);  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.
- * q, k float [rows, kv_heads * dim] (head h uses q/k head h / (heads / kv_heads)), v and o float [rows, heads * vdim].
+ * q, k float [rows, kv_heads * dim] (heads / kv_heads neighbouring heads share one q and k), v and o float [rows, heads * vdim].
  * per_channel 0: a at column a_col + head, dt_bias [heads]; 1: a at a_col + head * dim + channel, dt_bias [heads * dim].
  * a and b are float sources; state float [heads, dim, vdim] per slot.  dim <= 256. */
 NS_API int ns_delta_recurrent(ns_device_t dev, uint64_t q, int q_ld, uint64_t k, int k_ld, uint64_t v, int v_ld, uint64_t a_src, int a_splits, int a_ld,
@@ -492,7 +492,7 @@ NS_API int ns_latent_gather(ns_device_t dev, uint64_t ring, int64_t ring_slot_st
                             int rows, uint64_t keys);
 /* Windowed causal attention of a portion of `steps` tokens whose keys and values are expanded: q bf16 [rows, heads * (dim +
  * rot_dim)] (rotated), kv bf16 [batch * (past + steps), heads * dim keys | heads * vdim values], keys as ns_latent_gather leaves
- * them (the rotated key part, shared by all heads, at column rank), o bf16 [rows, heads * vdim]. */
+ * them (one rotated part for all heads, at column rank), o bf16 [rows, heads * vdim]. */
 NS_API int ns_latent_prefill(ns_device_t dev, uint64_t q, int64_t q_ld, uint64_t kv, int64_t kv_ld, uint64_t keys, int64_t keys_ld, int rank, uint64_t slots,
                              uint64_t pos, int batch, int steps, int heads, int dim, int rot_dim, int vdim, int past, int window, float scale, uint64_t o,
                              int64_t o_ld);

@@ -203,7 +203,7 @@ class DeltaMixer:
     """Gated delta rule with short convolutions (ns_delta.cu, ns_delta_chunk.cu).
 
     weights: q, k, v, b, o, their convolutions q_conv, k_conv, v_conv, A_log, dt_bias, norm, and either a, g (one decay per head,
-    read-out gated by silu) or a1, a2, g1, g2 (one decay per head and key channel through a low-rank pair, read-out gated by the
+    read-out gated by silu) or a1, a2, g1, g2 (a decay for every key channel of a head through a low-rank pair, read-out gated by the
     sigmoid of another).
 
     A few tokens go through the recurrence one by one, a prompt's portion (bf16 models) in chunks on the tensor cores; the choice

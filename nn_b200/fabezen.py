@@ -3,8 +3,8 @@ attention over a sliding window, in any order, with a bigram embedding and a tie
 
 The model is a list of blocks (nn_b200.blocks) over a 32-bit residual stream:
     x <- x + m * mixer(rms(x));  x <- x + m * ff(rms(x))
-and the row kernel that adds a block's output also normalises for the next block.  A layer may use another layer's weights with a
-cache and state of its own.  Sequences live in slots (nn_b200.state); there is no limit on a sequence's length, because windows
+and the row kernel that adds a block's output also normalises for the next block.  Layers may share weights; what
+a sequence carries is kept per layer.  Sequences live in slots (nn_b200.state); there is no limit on a sequence's length, because windows
 are rings and the other layers are recurrent.
 """
 from __future__ import annotations

@@ -1,8 +1,8 @@
 """Replays a trace: token ids fed through a model step by step, logits written where they are asked for; nothing is sampled.
 
 Steps come as JSON lines: {"step": n, "entries": [{"id", "tokens", "want"}], "end": [ids]}.  An entry's tokens continue what its
-id was fed before; "want" names places among them.  For a step that wants something, <out>/<n>.f32 holds the logits in the order
-of the entries and their "want", little-endian 32-bit floats; after every step the line "done <n>" is printed.
+id was fed before; "want" names places among them.  A step that wants something leaves <out>/<n>.f32: one row of
+little-endian 32-bit floats per wanted place, entry by entry; "done <n>" on standard output marks a step's end.
 """
 from __future__ import annotations
 
