@@ -367,6 +367,7 @@ __global__ void __launch_bounds__(256, MT == 1 && NW <= 8 ? 2 : 1) ns_latent_dec
         ns_fence_barrier_init();
         ns_fence_proxy_async();
     }
+    __syncthreads();
     ns_pdl_wait();
     ns_pdl_trigger();
     const int b = blockIdx.z, row0 = blockIdx.y * R, split = blockIdx.x;
@@ -376,17 +377,6 @@ __global__ void __launch_bounds__(256, MT == 1 && NW <= 8 ? 2 : 1) ns_latent_dec
     const int tiles = (last - first) / DC_KEYS + 1, per = (tiles + a.splits - 1) / a.splits;
     const int tb = split * per, te = min(tiles, tb + per);
 
-    for (int r = warp; r < R; r += 8) {
-        const bool in = row0 + r < a.rows;
-        const uint16_t* src = a.q + ((int64_t)b * a.rows + (in ? row0 + r : 0)) * a.width;
-        for (int c = lane * 8; c < a.wp; c += 256) ns_copy8(sQ + (r * ld + c) * 2, src + (c < a.width ? c : 0), in ? a.width - c : 0, (a.width & 7) == 0);
-    }
-    // columns past the cached row stay zero
-    for (int r = warp; r < 2 * DC_KEYS; r += 8)
-        for (int c = a.ring_ld + lane * 8; c < a.wp; c += 256) ns_st_shared_v4(sC + (r * ld + c) * 2, 0, 0, 0, 0);
-    ns_cp_commit();
-    ns_cp_wait<0>();
-    __syncthreads();
     // Warp 0 orders the rows of a tile as one bulk copy each; rows past the last position become zero.
     auto load_tile = [&](int t, int stage) {
         const int p0 = first + t * DC_KEYS, count = min(DC_KEYS, last - p0 + 1);
@@ -401,6 +391,19 @@ __global__ void __launch_bounds__(256, MT == 1 && NW <= 8 ? 2 : 1) ns_latent_dec
                 for (int c = lane * 8; c < a.ring_ld; c += 256) ns_st_shared_v4(sC + ((stage * DC_KEYS + r) * ld + c) * 2, 0, 0, 0, 0);
         }
     };
+    if (tb < te) load_tile(tb, 0);
+
+    for (int r = warp; r < R; r += 8) {
+        const bool in = row0 + r < a.rows;
+        const uint16_t* src = a.q + ((int64_t)b * a.rows + (in ? row0 + r : 0)) * a.width;
+        for (int c = lane * 8; c < a.wp; c += 256) ns_copy8(sQ + (r * ld + c) * 2, src + (c < a.width ? c : 0), in ? a.width - c : 0, (a.width & 7) == 0);
+    }
+    // columns past the cached row stay zero
+    for (int r = warp; r < 2 * DC_KEYS; r += 8)
+        for (int c = a.ring_ld + lane * 8; c < a.wp; c += 256) ns_st_shared_v4(sC + (r * ld + c) * 2, 0, 0, 0, 0);
+    ns_cp_commit();
+    ns_cp_wait<0>();
+    __syncthreads();
 
     float acc[MT][NW][4];
 #pragma unroll
@@ -414,7 +417,6 @@ __global__ void __launch_bounds__(256, MT == 1 && NW <= 8 ? 2 : 1) ns_latent_dec
 #pragma unroll
     for (int i = 0; i < 2 * MT; i++) { m[i] = -INFINITY; l[i] = 0.0f; }
 
-    if (tb < te) load_tile(tb, 0);
     for (int t = tb; t < te; t++) {
         const int stage = (t - tb) & 1;
         if (t + 1 < te) load_tile(t + 1, stage ^ 1);
