@@ -48,7 +48,7 @@ enum {
 };
 
 /* Activation of a gate. */
-enum { NS_ACT_SILU = 0, NS_ACT_SIGMOID = 1 };
+enum { NS_ACT_SILU = 0, NS_ACT_SIGMOID = 1, NS_ACT_GELU = 2, NS_ACT_RELU = 3 };
 
 /* How a Linear layer is divided among tensor-parallel ranks. */
 enum { NS_SPLIT_NONE = 0, NS_SPLIT_COLUMN = 1, NS_SPLIT_ROW = 2 };
@@ -427,8 +427,12 @@ NS_API int ns_embed_ngram(ns_device_t dev, uint64_t ids, uint64_t table, int tab
  * row_map[r]; src_rows is the number of rows of the source. */
 NS_API int ns_rms_rows(ns_device_t dev, uint64_t x, uint64_t src, int splits, int src_dtype, int src_ld, float alpha, uint64_t x_out, uint64_t w, float eps,
                        uint64_t row_map, int64_t src_rows, int64_t rows, int cols, int out_dtype, uint64_t y, int y_ld);
-/* y[r, c] = gelu_tanh(source[r, c]) * source[r, ff + c] */
-NS_API int ns_glu_rows(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int64_t rows, int ff, int out_dtype, uint64_t y, int y_ld);
+/* The residual update of layers that normalise a sublayer's output too: x_out = x + source / sqrt(mean(source^2) + eps) * post_w
+ * (+ plus, float [rows, cols], may be 0), x_out may be x; then, when w != 0, y = x_out / sqrt(mean(x_out^2) + eps) * w of out_dtype. */
+NS_API int ns_rms_post_rows(ns_device_t dev, uint64_t x, uint64_t src, int splits, int src_dtype, int src_ld, uint64_t post_w, uint64_t plus, uint64_t x_out, uint64_t w,
+                            float eps, int64_t rows, int cols, int out_dtype, uint64_t y, int y_ld);
+/* y[r, c] = act(source[r, c]) * source[r, ff + c], act NS_ACT_GELU (tanh form) or NS_ACT_RELU */
+NS_API int ns_glu_rows(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int64_t rows, int ff, int act, int out_dtype, uint64_t y, int y_ld);
 /* y[r, 0:cols] = source[r, col:col+cols] in another type or pitch */
 NS_API int ns_copy_cols(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int col, int64_t rows, int cols, int out_dtype, uint64_t y,
                         int y_ld);
@@ -459,10 +463,49 @@ NS_API int ns_delta_chunked(ns_device_t dev, uint64_t q, int q_ld, uint64_t k, i
                             int a_col, uint64_t b_src, int b_splits, int b_ld, int b_col, uint64_t a_log, uint64_t dt_bias, int per_channel,
                             uint64_t state, int64_t state_slot_stride, uint64_t slots, int batch, int steps, int heads, int kv_heads, int dim, int vdim,
                             uint64_t o, int o_ld);
-/* Per row and head: y = o / sqrt(mean(o^2) + eps) * w * act(gate), act NS_ACT_*; w float [vdim], gate at column gate_col of a
+/* Per row and head: y = o / sqrt(mean(o^2) + eps) * w * act(gate), act NS_ACT_SILU or NS_ACT_SIGMOID; w float [vdim], gate at column gate_col of a
  * source, y [rows, heads * vdim] of out_dtype. */
 NS_API int ns_gated_norm(ns_device_t dev, uint64_t o, int o_ld, uint64_t gate, int splits, int gate_dtype, int gate_ld, int gate_col, int act, uint64_t w,
                          float eps, int64_t rows, int heads, int vdim, int out_dtype, uint64_t y, int y_ld);
+
+/* Linear attention with one fixed decay per head, token by token: q, k = silu of the source's columns q_col, k_col + head * dim,
+ * v = silu of v_col + head * vdim;  S <- decay S + k v^T;  o = S^T q.  state: slot 0's float [heads, dim, vdim]; decay float [heads],
+ * decay_log2 its base-2 logarithms (finite: a decay of 0 as a large negative number); o float [rows, heads * vdim].  dim <= 256. */
+NS_API int ns_lightning_recurrent(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int q_col, int k_col, int v_col, uint64_t decay,
+                                  uint64_t decay_log2, uint64_t state, int64_t state_slot_stride, uint64_t slots, int batch, int steps, int heads, int dim,
+                                  int vdim, uint64_t o, int o_ld);
+/* The same for a prompt's portion, 64 tokens at a time on the tensor cores: q, k, v rounded to bf16 after the activation, state, decays
+ * and sums 32-bit (two bf16 halves as operands).  dim <= 128.  segments: pieces of a sequence that run side by side (0: chosen by the
+ * number of CTAs; bf16 sources only, their states lie in the device object's scratch block). */
+NS_API int ns_lightning_chunked(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int q_col, int k_col, int v_col, uint64_t decay,
+                                uint64_t decay_log2, uint64_t state, int64_t state_slot_stride, uint64_t slots, int batch, int steps, int heads, int dim,
+                                int vdim, uint64_t o, int o_ld, int segments);
+
+/* Grouped-query attention over a sliding window.  The cache of a sequence is a ring of keys [kv_heads, ring_len, k_ld] and one of
+ * values [kv_heads, ring_len, v_ld] (slot 0's address and the stride between slots, in elements), position p in row p modulo
+ * ring_len; ring_len is a multiple of 128 and at least window - 1 + steps, k_ld and v_ld are multiples of 8; the rings start
+ * as zeros.  append: q = RMS norm of the source's columns q_col, heads * dim of them together, with q_norm (0: as they are), in
+ * rows [heads, k_ld] padded with zeros; keys likewise with k_norm, and values, to the rings; gate[row, head] (float, may be 0) =
+ * sigmoid of column g_col + head. */
+NS_API int ns_window_append(ns_device_t dev, uint64_t src, int splits, int src_dtype, int src_ld, int q_col, int k_col, int v_col, int g_col, int heads, int kv_heads,
+                            int dim, int vdim, uint64_t q_norm, uint64_t k_norm, float eps, uint64_t slots, uint64_t pos, int batch, int steps, int dtype,
+                            uint64_t q, uint64_t gate, uint64_t k_ring, uint64_t v_ring, int64_t k_slot_stride, int64_t v_slot_stride, int ring_len, int k_ld,
+                            int v_ld);
+/* o[row, head, :] = gate[row, head] * sum_j e^(scale q . k_j) v_j / (e^sink[head] + sum_j e^(scale q . k_j)) over the positions j with
+ * 0 <= i - j < window; sink float [heads] and gate may be 0.  32-bit throughout, rings and o of dtype; any number of tokens. */
+NS_API int ns_window_attend(ns_device_t dev, int dtype, uint64_t q, uint64_t k_ring, uint64_t v_ring, int64_t k_slot_stride, int64_t v_slot_stride, int ring_len,
+                            int k_ld, int v_ld, uint64_t sink, uint64_t gate, uint64_t slots, uint64_t pos, int batch, int steps, int heads, int kv_heads, int dim,
+                            int vdim, int window, float scale, uint64_t o, int64_t o_ld);
+/* The same in bf16 on the tensor cores for few tokens (k_ld, v_ld <= 256): the query heads of a key/value head share its rows' read.
+ * Uses the device object's scratch block when the window is split over CTAs. */
+NS_API int ns_window_decode(ns_device_t dev, uint64_t q, uint64_t k_ring, uint64_t v_ring, int64_t k_slot_stride, int64_t v_slot_stride, int ring_len, int k_ld,
+                            int v_ld, uint64_t sink, uint64_t gate, uint64_t slots, uint64_t pos, int batch, int steps, int heads, int kv_heads, int dim, int vdim,
+                            int window, float scale, uint64_t o, int64_t o_ld);
+/* The same for a prompt's portion, by the kernel of ns_attention_prefill: k_ld, v_ld <= 128, vdim and o_ld multiples of 8, scale > 0;
+ * slot_count is the number of slots behind the rings' addresses. */
+NS_API int ns_window_prefill(ns_device_t dev, uint64_t q, uint64_t k_ring, uint64_t v_ring, int64_t k_slot_stride, int64_t v_slot_stride, int slot_count, int ring_len,
+                             int k_ld, int v_ld, uint64_t sink, uint64_t gate, uint64_t slots, uint64_t pos, int batch, int steps, int heads, int kv_heads, int dim,
+                             int vdim, int window, float scale, uint64_t o, int64_t o_ld);
 
 /* A row of the source is [query latent q_rank | latent kv_rank | rotated key part rot_dim].  cq = RMS norm of the first with
  * q_norm; the cache row of the token's position (ring row = position modulo ring_len) = [RMS norm of the second with kv_norm |

@@ -177,11 +177,18 @@ def rms_rows(step: Step, dev: Device, x: int, source: Source | None, alpha: floa
     step.launches += 1
 
 
-class DenseGlu:
-    """W_down (gelu_tanh(W_gate h) * (W_up h))."""
+def rms_post_rows(step: Step, dev: Device, x: int, source: Source, post, plus: int, x_out: int, weight, eps: float, cols: int, y: int, dtype: int, y_ld: int) -> None:
+    """x_out = x + RMS norm of the source with `post` (+ the rows at `plus`); y = RMS norm of it (weight None: no norm)."""
+    N.call("ns_rms_post_rows", dev.handle, C.c_uint64(x), *source.args, C.c_uint64(post.ptr), C.c_uint64(plus), C.c_uint64(x_out),
+           C.c_uint64(weight.ptr if weight else 0), C.c_float(eps), C.c_int64(step.m), cols, dtype, C.c_uint64(y), y_ld)
+    step.launches += 1
 
-    def __init__(self, ws: Workspace, gate, up, down):
-        self.dev, self.ws = ws.dev, ws
+
+class DenseGlu:
+    """W_down (act(W_gate h) * (W_up h)), act gelu (tanh form) or relu."""
+
+    def __init__(self, ws: Workspace, gate, up, down, act: int = N.ACT_GELU):
+        self.dev, self.ws, self.act = ws.dev, ws, act
         self.ff = gate.shape[0]
         self.gate_up = Product(ws, gate, up, wide=True)
         self.down = Product(ws, down)
@@ -190,7 +197,8 @@ class DenseGlu:
     def forward(self, h: int, step: Step) -> Source:
         s = self.gate_up.wide(h, step)
         act = self.ws["act"]
-        N.call("ns_glu_rows", self.dev.handle, *s.args, C.c_int64(step.m), self.ff, self.ws.dtype, C.c_uint64(act), self.down.k_ld)
+        N.call("ns_glu_rows", self.dev.handle, *s.args, C.c_int64(step.m), self.ff, self.act, self.ws.dtype, C.c_uint64(act),
+               self.down.k_ld)
         step.launches += 1
         return self.down(act, step)
 
@@ -290,6 +298,128 @@ class DeltaMixer:
         for p in (self.inputs, self.second, self.small, self.out):
             if p is not None:
                 p.close()
+
+
+class LightningMixer:
+    """Linear attention with a fixed decay per head (ns_lightning.cu): q, k, v through silu, the heads' outputs normalised together, times a
+    sigmoid gate per channel.
+
+    weights: q, k, v, g, o, norm.
+
+    A few tokens go through the recurrence one by one, a prompt's portion (bf16 models) in chunks on the tensor cores; the choice
+    depends on the portion's length alone."""
+
+    CHUNK_STEPS = 16         # portions of at least this many tokens are chunked
+
+    def __init__(self, ws: Workspace, heads: int, dim: int, vdim: int, decay, eps: float, w: dict):
+        decay = np.asarray(decay, np.float64)
+        if decay.shape != (heads,) or not np.all(decay >= 0.0):
+            raise ValueError(f"{heads} heads need {heads} decays that are not negative")
+        self.dev, self.ws, self.eps = ws.dev, ws, eps
+        self.heads, self.dim, self.vdim = heads, dim, vdim
+        self.chunks = ws.dtype == N.NS_BF16 and dim <= 128
+        with np.errstate(divide="ignore"):
+            log2 = np.maximum(np.log2(decay), -1e4)          # a decay of 0: powers of it are 0 (and its 0th power 1)
+        up = lambda a: self.dev.from_numpy(np.ascontiguousarray(a, np.float32).reshape(-1))
+        self.decay, self.decay_log2, self.norm = up(decay), up(log2), up(f32(w["norm"]))
+        self.inputs = Product(ws, w["q"], w["k"], w["v"], w["g"], wide=True)
+        self.out = Product(ws, w["o"])
+        ws.need("read", heads * vdim, N.NS_F32)
+        ws.need("mixed", self.out.k_ld)
+
+    def reserve(self, states: SequenceStates, max_steps: int) -> Reservation:
+        return states.reserve(self.heads * self.dim * self.vdim, N.NS_F32, True)
+
+    def forward(self, h: int, cache: Reservation, step: Step) -> Source:
+        ws, hd, u = self.ws, self.dev.handle, C.c_uint64
+        s, n = self.inputs.wide(h, step), self.heads * self.vdim
+        q, k, v, g = self.inputs.cols
+        args = (hd, *s.args, q, k, v, u(self.decay.ptr), u(self.decay_log2.ptr), u(cache.ptr), C.c_int64(cache.stride), u(step.slots), step.batch, step.steps, self.heads,
+                self.dim, self.vdim, u(ws["read"]), n)
+        if self.chunks and step.steps >= self.CHUNK_STEPS:
+            N.call("ns_lightning_chunked", *args, 0)
+        else:
+            N.call("ns_lightning_recurrent", *args)
+        N.call("ns_gated_norm", hd, u(ws["read"]), n, *s.args, g, N.ACT_SIGMOID, u(self.norm.ptr), C.c_float(self.eps), C.c_int64(step.m), 1, n, ws.dtype,
+               u(ws["mixed"]), self.out.k_ld)
+        step.launches += 2
+        return self.out(ws["mixed"], step)
+
+    def close(self) -> None:
+        self.inputs.close()
+        self.out.close()
+
+
+class WindowAttentionMixer:
+    """Grouped-query attention over a sliding window (ns_window.cu; a prompt's portion: ns_attention_prefill.cu).
+
+    weights: q, k, v, o, and, each optional, q_norm and k_norm (RMS norm over all heads together), sink (a learned term of every
+    head's softmax sum), g (a sigmoid gate per head on its output).
+
+    Portions of a few tokens and longer ones take different kernels; the choice depends on the portion's length alone."""
+
+    PREFILL_STEPS = 32       # portions of at least this many tokens are a prompt's
+    RING_ROWS = 128          # ring lengths are multiples of this
+
+    def __init__(self, ws: Workspace, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, eps: float, w: dict):
+        if heads % kv_heads != 0:
+            raise ValueError(f"{heads} heads do not divide over {kv_heads} key/value heads")
+        if window < 1:
+            raise ValueError(f"a window of {window} positions")
+        self.dev, self.ws, self.eps, self.window = ws.dev, ws, eps, window
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.k_ld, self.v_ld = pad8(dim), pad8(vdim)
+        bf16 = ws.dtype == N.NS_BF16
+        self.tiles = bf16 and self.k_ld <= 256 and self.v_ld <= 256
+        self.prefill = bf16 and self.k_ld <= 128 and self.v_ld <= 128 and vdim % 8 == 0
+        up = lambda name, sign=1.0: self.dev.from_numpy(f32(w[name]).reshape(-1) * np.float32(sign)) if w.get(name) is not None else None
+        # the kernels take a positive scale: the queries carry its sign
+        sign = 1.0 if scale > 0.0 else (-1.0 if scale < 0.0 else 0.0)
+        self.scale = abs(scale) or 1.0
+        q = w["q"]
+        if sign != 1.0 and w.get("q_norm") is None:
+            q, sign = f32(q) * np.float32(sign), 1.0
+        self.q_norm, self.k_norm, self.sink = up("q_norm", sign), up("k_norm"), up("sink")
+        self.gated = w.get("g") is not None
+        self.inputs = Product(ws, q, w["k"], w["v"], *((w["g"],) if self.gated else ()), wide=True)
+        self.out = Product(ws, w["o"])
+        ws.need("q_heads", heads * self.k_ld)
+        if self.gated:
+            ws.need("gate", heads, N.NS_F32)
+        # the columns that pad a row of the output product's input are never written: a buffer of this width's own keeps them zero
+        self.mixed = f"mixed_{heads * vdim}"
+        ws.need(self.mixed, self.out.k_ld)
+
+    def reserve(self, states: SequenceStates, max_steps: int) -> dict:
+        """The rings are cleared when a sequence opens: the kernels read whole tiles of rows and mask by position, so every row has to be finite."""
+        n = -(-(self.window - 1 + max_steps) // self.RING_ROWS) * self.RING_ROWS
+        return {"k": states.reserve(self.kv_heads * n * self.k_ld, self.ws.dtype, True), "v": states.reserve(self.kv_heads * n * self.v_ld, self.ws.dtype, True),
+                "len": n, "slots": states.slots}
+
+    def forward(self, h: int, cache: dict, step: Step) -> Source:
+        ws, hd, u, i64 = self.ws, self.dev.handle, C.c_uint64, C.c_int64
+        k, v = cache["k"], cache["v"]
+        rings = (u(k.ptr), u(v.ptr), i64(k.stride), i64(v.stride))
+        lens = (cache["len"], self.k_ld, self.v_ld)
+        at = (u(step.slots), u(step.pos), step.batch, step.steps)
+        s, cols = self.inputs.wide(h, step), self.inputs.cols
+        q, gate, mixed = u(ws["q_heads"]), u(ws["gate"] if self.gated else 0), u(ws[self.mixed])
+        ptr = lambda a: u(a.ptr if a is not None else 0)
+        N.call("ns_window_append", hd, *s.args, cols[0], cols[1], cols[2], cols[3] if self.gated else 0, self.heads, self.kv_heads, self.dim, self.vdim,
+               ptr(self.q_norm), ptr(self.k_norm), C.c_float(self.eps), *at, ws.dtype, q, gate, *rings, *lens)
+        rest = (ptr(self.sink), gate, *at, self.heads, self.kv_heads, self.dim, self.vdim, self.window, C.c_float(self.scale), mixed, i64(self.out.k_ld))
+        if self.prefill and step.steps >= self.PREFILL_STEPS:
+            N.call("ns_window_prefill", hd, q, *rings, cache["slots"], *lens, *rest)
+        elif self.tiles:
+            N.call("ns_window_decode", hd, q, *rings, *lens, *rest)
+        else:
+            N.call("ns_window_attend", hd, ws.dtype, q, *rings, *lens, *rest)
+        step.launches += 2
+        return self.out(ws[self.mixed], step)
+
+    def close(self) -> None:
+        self.inputs.close()
+        self.out.close()
 
 
 class LatentAttentionMixer:

@@ -30,6 +30,12 @@
 //               the 128 output dims through shared memory with TMA stores.
 // Tensor memory: S_0 at columns [0,128), S_1 at [128,256), O_0 at [256,384), O_1 at [384,512).
 // Every mbarrier wait is bounded; a wait that runs out reports a status code and the CTA leaves.
+//
+// The same kernel serves a portion of a prompt against the rings of a sliding window (ns_window_prefill; ns_window.cu has the rings and
+// the form for few tokens): key blocks are then the 128 positions from a multiple of 128 on, only those that the window of
+// one of the tile's rows reaches are walked, several query heads may share a key/value head, heads have up to 128 columns (the
+// maps fill the rest with zeros; up to 64 use one half), and where the two groups' results are merged a row's sink joins its
+// sum and its gate its result.
 #include <math.h>
 
 #include "ns_common.cuh"
@@ -48,6 +54,12 @@ struct FaParams {
     float scale_log2;  // scale * log2(e)
     int* status;
     int* tile_counter; // zeroed before the launch: CTAs draw their tiles from it in order
+    // windowed form: seq counts the portion's tokens, which follow pos[slots[b]] earlier ones
+    int window, ring_len, kv_share;   // kv_share: query heads per key/value head
+    const int32_t* slots;
+    const int32_t* pos;
+    const float* sink;                // [heads] or null
+    const float* gate;                // [batch * seq, heads] or null
 };
 
 struct FaMaps {
@@ -77,7 +89,9 @@ enum { BAR_Q = 0, BAR_Q_FREE = 1, BAR_K0 = 2, BAR_V0 = 4, BAR_K_EMPTY0 = 6, BAR_
 // but the first reader hit in L2, and whichever CTA is free takes the next tile, so the CTAs finish together.
 struct FaTile {
     int b, h, q0, n_blocks;
+    int pos0, j0;      // windowed form: the sequence's earlier tokens, the first key block
 };
+template <bool WINDOW>
 __device__ __forceinline__ void fa_tile(const FaParams& p, int n_qt, int idx, FaTile& t)
 {
     const int qt = n_qt - 1 - idx % n_qt;
@@ -86,8 +100,18 @@ __device__ __forceinline__ void fa_tile(const FaParams& p, int n_qt, int idx, Fa
     t.h = bh % p.heads;
     t.q0 = qt * FA_BLOCK;
     t.n_blocks = p.causal ? qt + 1 : n_qt;
+    if (WINDOW) t.j0 = 0;
+}
+// the key blocks that the windows of the tile's rows reach
+__device__ __forceinline__ void fa_window(const FaParams& p, int pos0, FaTile& t)
+{
+    t.pos0 = pos0;
+    t.j0 = max(0, pos0 + t.q0 - p.window + 1) / FA_BLOCK;
+    t.n_blocks = (pos0 + min(t.q0 + FA_BLOCK, p.seq) - 1) / FA_BLOCK - t.j0 + 1;
 }
 
+// KH, VH: 64-column halves of a query / key and of a value
+template <int KH, int VH, bool WINDOW>
 __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(const __grid_constant__ FaMaps maps, const FaParams p)
 {
     extern __shared__ uint8_t smem_raw[];
@@ -113,9 +137,17 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
     auto next_tile = [&](int it, FaTile& t) {
         if (!ns_mbar_wait(bar(BAR_TILE0 + (it & 3)), (it >> 2) & 1, abort_flag, p.status, 300 + 11)) return false;
         int idx;
+        if (WINDOW) {
+            int pos0;
+            asm volatile("ld.shared.v2.b32 {%0, %1}, [%2];" : "=r"(idx), "=r"(pos0) : "r"(tile_ring + 8u * (it & 3)) : "memory");
+            if (idx < 0) return false;
+            fa_tile<WINDOW>(p, n_qt, idx, t);
+            fa_window(p, pos0, t);
+            return true;
+        }
         asm volatile("ld.shared.b32 %0, [%1];" : "=r"(idx) : "r"(tile_ring + 4u * (it & 3)) : "memory");
         if (idx < 0) return false;
-        fa_tile(p, n_qt, idx, t);
+        fa_tile<WINDOW>(p, n_qt, idx, t);
         return true;
     };
 
@@ -162,20 +194,23 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
     if (warp == 0) {
         // ------------------------------------------------------------ producer
         if (lane == 0) {
+            // where block j's rows, and the head, lie in the maps
+            int slot = 0, pos0 = 0, seq_now = -1;
+            auto key_row = [&](const FaTile& t, int j) { return WINDOW ? (t.j0 + j) * FA_BLOCK % p.ring_len : j * FA_BLOCK; };
             auto load_k = [&](const FaTile& t, int j, int gj) {
-                const int s = gj & 1;
+                const int s = gj & 1, y = key_row(t, j), z = WINDOW ? t.h / p.kv_share : t.h, w = WINDOW ? slot : t.b;
                 if (gj >= 2 && !ns_mbar_wait(bar(BAR_K_EMPTY0 + s), ((gj >> 1) - 1) & 1, abort_flag, p.status, code + 1)) return false;
-                ns_mbar_expect_tx(bar(BAR_K0 + s), FA_TILE_BYTES);
-                ns_tma_load_4d(k_smem(s), &maps.k, bar(BAR_K0 + s), 0, j * FA_BLOCK, t.h, t.b);
-                ns_tma_load_4d(k_smem(s) + FA_HALF_BYTES, &maps.k, bar(BAR_K0 + s), 64, j * FA_BLOCK, t.h, t.b);
+                ns_mbar_expect_tx(bar(BAR_K0 + s), KH * FA_HALF_BYTES);
+#pragma unroll
+                for (int i = 0; i < KH; i++) ns_tma_load_4d(k_smem(s) + i * FA_HALF_BYTES, &maps.k, bar(BAR_K0 + s), i * 64, y, z, w);
                 return true;
             };
             auto load_v = [&](const FaTile& t, int j, int gj) {
-                const int s = gj & 1;
+                const int s = gj & 1, y = key_row(t, j), z = WINDOW ? t.h / p.kv_share : t.h, w = WINDOW ? slot : t.b;
                 if (gj >= 2 && !ns_mbar_wait(bar(BAR_V_EMPTY0 + s), ((gj >> 1) - 1) & 1, abort_flag, p.status, code + 1)) return false;
-                ns_mbar_expect_tx(bar(BAR_V0 + s), FA_TILE_BYTES);
-                ns_tma_load_4d(v_smem(s), &maps.v, bar(BAR_V0 + s), 0, j * FA_BLOCK, t.h, t.b);
-                ns_tma_load_4d(v_smem(s) + FA_HALF_BYTES, &maps.v, bar(BAR_V0 + s), 64, j * FA_BLOCK, t.h, t.b);
+                ns_mbar_expect_tx(bar(BAR_V0 + s), VH * FA_HALF_BYTES);
+#pragma unroll
+                for (int i = 0; i < VH; i++) ns_tma_load_4d(v_smem(s) + i * FA_HALF_BYTES, &maps.v, bar(BAR_V0 + s), i * 64, y, z, w);
                 return true;
             };
             bool ok = true;
@@ -186,13 +221,26 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
                 if (it > 0) ok = ns_mbar_wait(bar(BAR_Q_FREE), (it - 1) & 1, abort_flag, p.status, code + 1);
                 if (!ok) break;
                 const int idx = atomicAdd(p.tile_counter, 1);
-                asm volatile("st.shared.b32 [%0], %1;" ::"r"(tile_ring + 4u * (it & 3)), "r"(idx < total ? idx : -1) : "memory");
+                if (WINDOW) {
+                    if (idx < total) {
+                        fa_tile<WINDOW>(p, n_qt, idx, t);
+                        if (t.b != seq_now) {            // the tiles of a sequence follow one another
+                            seq_now = t.b;
+                            slot = p.slots[t.b];
+                            pos0 = p.pos[slot];
+                        }
+                        fa_window(p, pos0, t);
+                    }
+                    asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(tile_ring + 8u * (it & 3)), "r"(idx < total ? idx : -1), "r"(pos0) : "memory");
+                } else {
+                    asm volatile("st.shared.b32 [%0], %1;" ::"r"(tile_ring + 4u * (it & 3)), "r"(idx < total ? idx : -1) : "memory");
+                }
                 ns_mbar_arrive(bar(BAR_TILE0 + (it & 3)));
                 if (idx >= total) break;
-                fa_tile(p, n_qt, idx, t);
-                ns_mbar_expect_tx(bar(BAR_Q), FA_TILE_BYTES);
-                ns_tma_load_4d(q_smem, &maps.q, bar(BAR_Q), 0, t.q0, t.h, t.b);
-                ns_tma_load_4d(q_smem + FA_HALF_BYTES, &maps.q, bar(BAR_Q), 64, t.q0, t.h, t.b);
+                if (!WINDOW) fa_tile<WINDOW>(p, n_qt, idx, t);
+                ns_mbar_expect_tx(bar(BAR_Q), KH * FA_HALF_BYTES);
+#pragma unroll
+                for (int i = 0; i < KH; i++) ns_tma_load_4d(q_smem + i * FA_HALF_BYTES, &maps.q, bar(BAR_Q), i * 64, t.q0, t.h, t.b);
                 // K_j is wanted early (scores are computed two blocks ahead of the softmax), V_j late: K slots are freed by the
                 // Q.K^T that read them, V slots by the P.V, and V trails K by one block
                 for (int j = 0; j <= t.n_blocks && ok; j++) {
@@ -206,7 +254,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
         // ------------------------------------------------------------ MMA issuer
         if (lane == 0) {
             constexpr uint32_t idesc_qk = ns_idesc(1, 1, 0, 0, 128, 128);
-            constexpr uint32_t idesc_pv = ns_idesc(1, 1, 0, 1, 128, 128);
+            constexpr uint32_t idesc_pv = ns_idesc(1, 1, 0, 1, 128, VH * 64);
             const uint64_t desc_k = ns_desc_base(16, 1024);
             const uint64_t desc_v = ns_desc_base(FA_HALF_BYTES, 1024);  // MN-major: 64-dim halves 16 KB apart, 8 key rows 1 KB apart
             auto issue_qk = [&](int gj, bool last_of_tile) {
@@ -214,7 +262,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
                 const uint32_t d_tmem = tmem_base + s * 128;
                 const uint32_t kb = k_smem(s);
 #pragma unroll
-                for (int kk = 0; kk < 8; kk++) {
+                for (int kk = 0; kk < KH * 4; kk++) {
                     const uint32_t off = (kk >> 2) * FA_HALF_BYTES + (kk & 3) * 32;
                     ns_mma_f16(d_tmem, ns_desc_at(desc_k, q_smem + off), ns_desc_at(desc_k, kb + off), idesc_qk, kk > 0 ? 1u : 0u);
                 }
@@ -305,7 +353,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
         int kg = 0;                               // blocks this group has handled so far, over all tiles
         FaTile t;
         for (int it = 0; ok && next_tile(it, t); it++) {
-            const int qi = t.q0 + r;             // absolute query position
+            const int qi = WINDOW ? t.pos0 + t.q0 + r : t.q0 + r;   // absolute query position
             float m_ref = -INFINITY;             // reference maximum of this group's blocks of the tile (raw score units)
             float l_run = 0.0f;                  // sum of this group's exponentials relative to m_ref
             int n_mine = 0;
@@ -328,15 +376,17 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
                 ns_tc_fence_before();
                 ns_mbar_arrive(bar(BAR_S_FREE0 + g));
                 // mask: keys after the query (causal) or past the end of the sequence
-                const int kv0 = j * FA_BLOCK;
-                const bool need_mask = (p.causal && kv0 + 127 > t.q0) || kv0 + 128 > p.seq;
+                // windowed form: or more than the window before it (what a ring holds past a row's own position is later than it)
+                const int kv0 = (WINDOW ? t.j0 + j : j) * FA_BLOCK;
+                const bool need_mask = WINDOW ? kv0 + 127 > t.pos0 + t.q0 || kv0 <= t.pos0 + t.q0 + 127 - p.window
+                                              : (p.causal && kv0 + 127 > t.q0) || kv0 + 128 > p.seq;
                 float mx;
                 if (need_mask) {
                     mx = -INFINITY;
 #pragma unroll
                     for (int c = 0; c < 128; c++) {
                         const int kj = kv0 + c;
-                        const bool dead = (p.causal && kj > qi) || kj >= p.seq;
+                        const bool dead = WINDOW ? kj > qi || kj <= qi - p.window : (p.causal && kj > qi) || kj >= p.seq;
                         if (dead) sb[c] = 0xFF800000u;  // -inf
                         mx = fmaxf(mx, __uint_as_float(sb[c]));
                     }
@@ -381,7 +431,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
                     ns_tc_fence_after();
                     if (n_mine > 0 && __any_sync(0xffffffffu, rescale)) {
 #pragma unroll 1
-                        for (int c = 0; c < 4; c++) {
+                        for (int c = 0; c < 2 * VH; c++) {
                             uint32_t ob[32];
                             ns_tmem_ld32(o_addr + c * 32, ob);
                             ns_tc_wait_ld();
@@ -428,16 +478,28 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
             }
             if (ok) {
                 const float m_all = fmaxf(m_ref, m_o);
-                const float a_mine = m_ref == -INFINITY ? 0.0f : fa_exp2((m_ref - m_all) * p.scale_log2);
-                const float a_other = m_o == -INFINITY ? 0.0f : fa_exp2((m_o - m_all) * p.scale_log2);
+                float a_mine = m_ref == -INFINITY ? 0.0f : fa_exp2((m_ref - m_all) * p.scale_log2);
+                float a_other = m_o == -INFINITY ? 0.0f : fa_exp2((m_o - m_all) * p.scale_log2);
+                float l_sink = 0.0f, row_gate = 1.0f;
+                if (WINDOW) {
+                    if (p.sink != nullptr) {
+                        const float s = p.sink[t.h] * 1.4426950408889634f, m2 = m_all * p.scale_log2, top = fmaxf(m2, s), f = fa_exp2(m2 - top);
+                        l_sink = fa_exp2(s - top);
+                        a_mine *= f;
+                        a_other *= f;
+                    }
+                    if (p.gate != nullptr) row_gate = t.q0 + r < p.seq ? p.gate[((int64_t)t.b * p.seq + t.q0 + r) * p.heads + t.h] : 0.0f;
+                }
                 // Which group got the tile's even-numbered key blocks depends on how many blocks this CTA has walked before
                 // (tiles are drawn from a counter at run time).  The result must not: the two partial results are combined
                 // in the order (even blocks, odd blocks) of the TILE, whichever group holds which, with every rounding spelt out.
                 const bool mine_even = ((g - gj0) & 1) == 0;
                 const float l_even = mine_even ? l_run : l_o, a_even = mine_even ? a_mine : a_other;
                 const float l_odd = mine_even ? l_o : l_run, a_odd = mine_even ? a_other : a_mine;
-                const float l_tot = __fadd_rn(__fmul_rn(l_even, a_even), __fmul_rn(l_odd, a_odd));
-                const float inv = l_tot > 0.0f ? 1.0f / l_tot : 0.0f;
+                float l_tot = __fadd_rn(__fmul_rn(l_even, a_even), __fmul_rn(l_odd, a_odd));
+                if (WINDOW) l_tot = __fadd_rn(l_tot, l_sink);
+                float inv = l_tot > 0.0f ? 1.0f / l_tot : 0.0f;
+                if (WINDOW) inv *= row_gate;
                 const float w_even = __fmul_rn(a_even, inv), w_odd = __fmul_rn(a_odd, inv);
                 const uint32_t o_mine = lane_addr + 256 + g * 128, o_other = lane_addr + 256 + (g ^ 1) * 128;
                 // group g finishes output dims [64 g, 64 g + 64): (O_mine w_mine + O_other w_other) -> bf16 -> the upper half of
@@ -447,7 +509,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
                 const bool have_mine = n_mine > 0;
                 const bool have_other = t.n_blocks >= 2 || !have_mine;   // uniform over the CTA: the other group had a block
 #pragma unroll 1
-                for (int c = 0; c < 2; c++) {
+                for (int c = 0; c < 2 && g < VH; c++) {
                     uint32_t oa[32], ob[32];
 #pragma unroll
                     for (int q = 0; q < 32; q++) { oa[q] = 0u; ob[q] = 0u; }
@@ -476,7 +538,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
                 ns_mbar_arrive(bar(BAR_O_FREE));
                 ns_fence_proxy_async();
                 __syncwarp();
-                if (lane == 0 && t.q0 + quad * 32 < p.seq) {
+                if (lane == 0 && g < VH && t.q0 + quad * 32 < p.seq) {
                     ns_tma_store_4d(&maps.o, stage + quad * 32 * 128, g * 64, t.q0 + quad * 32, t.h, t.b);
                     ns_bulk_commit();
                     ns_bulk_wait_read<0>();
@@ -501,9 +563,9 @@ __global__ void __launch_bounds__(FA_THREADS, 1) ns_attention_prefill_kernel(con
     }
 }
 
-int make_map(CUtensorMap* m, uint64_t base, int batch, int heads, int seq, int64_t sb, int64_t sh, int64_t ss, uint32_t box_rows)
+int make_map(CUtensorMap* m, uint64_t base, int batch, int heads, int seq, int64_t sb, int64_t sh, int64_t ss, uint32_t box_rows, int cols = 128)
 {
-    uint64_t dims[4] = {128, (uint64_t)seq, (uint64_t)heads, (uint64_t)batch};
+    uint64_t dims[4] = {(uint64_t)cols, (uint64_t)seq, (uint64_t)heads, (uint64_t)batch};
     uint64_t strides[3] = {(uint64_t)ss * 2, (uint64_t)sh * 2, (uint64_t)sb * 2};
     uint32_t box[4] = {64, box_rows, 1, 1};
     return ns_make_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, reinterpret_cast<const void*>(base), dims, strides, box,
@@ -540,14 +602,69 @@ extern "C" int ns_attention_prefill(ns_device_t h, uint64_t q, uint64_t k, uint6
     p.batch = batch; p.heads = heads; p.seq = seq; p.causal = causal ? 1 : 0;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = d->status_dev;
+    p.window = p.ring_len = p.kv_share = 0;
+    p.slots = p.pos = nullptr;
+    p.sink = p.gate = nullptr;
     static bool configured[64] = {false};
     if (!configured[d->ordinal]) {
-        NS_CUDA(cudaFuncSetAttribute(ns_attention_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FA_SMEM_BYTES));
+        NS_CUDA(cudaFuncSetAttribute(ns_attention_prefill_kernel<2, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FA_SMEM_BYTES));
         configured[d->ordinal] = true;
     }
     // persistent: one CTA per SM walks its share of the (batch, head, query tile) list
     const int total = batch * heads * n_qt;
-    ns_attention_prefill_kernel<<<total < d->sm_count ? total : d->sm_count, FA_THREADS, FA_SMEM_BYTES, d->stream>>>(maps, p);
+    ns_attention_prefill_kernel<2, 2, false><<<total < d->sm_count ? total : d->sm_count, FA_THREADS, FA_SMEM_BYTES, d->stream>>>(maps, p);
     NS_CUDA(cudaGetLastError());
     return NS_OK;
+}
+
+template <int KH, int VH>
+static int launch_window(NsDevice* d, const FaMaps& maps, const FaParams& p, int total)
+{
+    auto k = ns_attention_prefill_kernel<KH, VH, true>;
+    NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FA_SMEM_BYTES));
+    k<<<total < d->sm_count ? total : d->sm_count, FA_THREADS, FA_SMEM_BYTES, d->stream>>>(maps, p);
+    NS_CUDA(cudaGetLastError());
+    return NS_OK;
+}
+
+extern "C" int ns_window_prefill(ns_device_t h, uint64_t q, uint64_t k_ring, uint64_t v_ring, int64_t k_slot_stride, int64_t v_slot_stride, int slot_count, int ring_len,
+                                 int k_ld, int v_ld, uint64_t sink, uint64_t gate, uint64_t slots, uint64_t pos, int batch, int steps, int heads, int kv_heads, int dim,
+                                 int vdim, int window, float scale, uint64_t o, int64_t o_ld)
+{
+    NsDevice* d = ns_dev(h);
+    int rc = ns_device_make_current(d);
+    if (rc != NS_OK) return rc;
+    NS_REQUIRE(q && k_ring && v_ring && slots && pos && o && batch > 0 && steps > 0 && slot_count > 0, NS_ERR_ARGUMENT, "ns_window_prefill: bad argument");
+    NS_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0, NS_ERR_ARGUMENT, "ns_window_prefill: %d heads do not divide over %d key/value heads", heads, kv_heads);
+    NS_REQUIRE(dim > 0 && dim <= k_ld && k_ld <= 128 && vdim > 0 && vdim <= v_ld && v_ld <= 128 && ((k_ld | v_ld | vdim) & 7) == 0 && (o_ld & 7) == 0 &&
+                   o_ld >= (int64_t)heads * vdim && ((k_slot_stride | v_slot_stride) & 7) == 0 && ((q | k_ring | v_ring | o) & 15) == 0,
+               NS_ERR_ARGUMENT, "ns_window_prefill: bad sizes");
+    NS_REQUIRE(scale > 0.0f, NS_ERR_ARGUMENT, "ns_window_prefill: the scale must be positive");
+    NS_REQUIRE(window > 0 && ring_len % FA_BLOCK == 0 && (int64_t)window - 1 + steps <= ring_len, NS_ERR_ARGUMENT,
+               "ns_window_prefill: a window of %d and %d tokens do not fit rings of %d rows (a multiple of 128)", window, steps, ring_len);
+    const int n_qt = (steps + FA_BLOCK - 1) / FA_BLOCK;
+    NS_REQUIRE((int64_t)batch * heads * n_qt < (1LL << 31), NS_ERR_ARGUMENT, "ns_window_prefill: too many tiles");
+    FaMaps maps;
+    rc = make_map(&maps.q, q, batch, heads, steps, (int64_t)steps * heads * k_ld, k_ld, (int64_t)heads * k_ld, 128, k_ld);
+    if (rc == NS_OK) rc = make_map(&maps.k, k_ring, slot_count, kv_heads, ring_len, k_slot_stride, (int64_t)ring_len * k_ld, k_ld, 128, k_ld);
+    if (rc == NS_OK) rc = make_map(&maps.v, v_ring, slot_count, kv_heads, ring_len, v_slot_stride, (int64_t)ring_len * v_ld, v_ld, 128, v_ld);
+    if (rc == NS_OK) rc = make_map(&maps.o, o, batch, heads, steps, (int64_t)steps * o_ld, vdim, o_ld, 32, vdim);
+    if (rc != NS_OK) return rc;
+    void* counter = nullptr;
+    rc = ns_scratch_reserve(d, 256, &counter);
+    if (rc != NS_OK) return rc;
+    NS_CUDA(cudaMemsetAsync(counter, 0, sizeof(int), d->stream));
+    FaParams p;
+    p.tile_counter = reinterpret_cast<int*>(counter);
+    p.batch = batch; p.heads = heads; p.seq = steps; p.causal = 1;
+    p.scale_log2 = scale * 1.4426950408889634f;
+    p.status = d->status_dev;
+    p.window = window; p.ring_len = ring_len; p.kv_share = heads / kv_heads;
+    p.slots = reinterpret_cast<const int32_t*>(slots);
+    p.pos = reinterpret_cast<const int32_t*>(pos);
+    p.sink = reinterpret_cast<const float*>(sink);
+    p.gate = reinterpret_cast<const float*>(gate);
+    const int total = batch * heads * n_qt;
+    if (k_ld <= 64) return v_ld <= 64 ? launch_window<1, 1>(d, maps, p, total) : launch_window<1, 2>(d, maps, p, total);
+    return v_ld <= 64 ? launch_window<2, 1>(d, maps, p, total) : launch_window<2, 2>(d, maps, p, total);
 }

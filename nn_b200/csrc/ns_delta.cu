@@ -426,6 +426,40 @@ __global__ void __launch_bounds__(256) ns_gated_norm_kernel(const float* __restr
     }
 }
 
+// The same for one wide head (the whole row): a CTA per row, up to 8 groups of four values per thread in registers.
+template <typename T, int Q>
+__global__ void __launch_bounds__(256) ns_gated_norm_row_kernel(const float* __restrict__ o, int o_ld, const NsSource gate, int gate_col, int act,
+                                                                const float* __restrict__ w, float eps, int n, T* __restrict__ y, int64_t y_ld)
+{
+    __shared__ float red[8];
+    ns_pdl_wait();
+    ns_pdl_trigger();
+    const int64_t row = blockIdx.x;
+    float4 v[Q], z[Q];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int c = (threadIdx.x + 256 * i) * 4;
+        v[i] = z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= n) continue;
+        v[i] = *reinterpret_cast<const float4*>(o + row * o_ld + c);
+        z[i] = ns_source_at4(gate, row * gate.ld + gate_col + c);
+    }
+#pragma unroll
+    for (int i = 0; i < Q; i++) { ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss); }
+    const float inv = 1.0f / sqrtf(ns_cta_sum(ss, red) / (float)n + eps);
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int c = (threadIdx.x + 256 * i) * 4;
+        if (c >= n) continue;
+        const float4 ww = __ldg(reinterpret_cast<const float4*>(w + c));
+        const float4 r = act == NS_ACT_SILU ? make_float4(ns_silu(z[i].x), ns_silu(z[i].y), ns_silu(z[i].z), ns_silu(z[i].w))
+                                            : make_float4(ns_sigmoid(z[i].x), ns_sigmoid(z[i].y), ns_sigmoid(z[i].z), ns_sigmoid(z[i].w));
+        ns_store4(y + row * y_ld + c, make_float4(v[i].x * inv * ww.x * r.x, v[i].y * inv * ww.y * r.y, v[i].z * inv * ww.z * r.z, v[i].w * inv * ww.w * r.w));
+    }
+    for (int c = n + threadIdx.x; c < y_ld; c += 256) ns_store(y + row * y_ld + c, 0.0f);
+}
+
 template <int RPW, int V>
 int launch_recurrent(NsDevice* d, const DeltaArgs& a, int batch, bool channel)
 {
@@ -571,7 +605,22 @@ extern "C" int ns_gated_norm(ns_device_t h, uint64_t o, int o_ld, uint64_t gate,
     NS_REQUIRE(act == NS_ACT_SILU || act == NS_ACT_SIGMOID, NS_ERR_ARGUMENT, "ns_gated_norm: unknown activation %d", act);
     NS_REQUIRE(out_dtype == NS_F32 || out_dtype == NS_BF16, NS_ERR_ARGUMENT, "ns_gated_norm: bad output type");
     const NsSource g = ns_source(gate, splits, gate_dtype, rows, gate_ld);
-    const bool vec = vdim <= 128 && ((vdim | o_ld | gate_ld | gate_col | y_ld) & 3) == 0 && ((o | gate | w | y) & 15) == 0;
+    const bool aligned = ((vdim | o_ld | gate_ld | gate_col | y_ld) & 3) == 0 && ((o | gate | w | y) & 15) == 0 && (g.slab & 3) == 0, vec = aligned && vdim <= 128;
+    if (aligned && heads == 1 && vdim > 128 && vdim <= 8192) {
+        auto row = [&](auto zero, auto kernel) -> int {
+            using T = decltype(zero);
+            NS_CUDA(ns_launch_plain(kernel, dim3((unsigned)rows), dim3(256), 0, d->stream, reinterpret_cast<const float*>(o), o_ld, g, gate_col, act,
+                                    reinterpret_cast<const float*>(w), eps, vdim, reinterpret_cast<T*>(y), (int64_t)y_ld));
+            return NS_OK;
+        };
+        auto pick = [&](auto zero) -> int {
+            using T = decltype(zero);
+            if (vdim <= 2048) return row(zero, ns_gated_norm_row_kernel<T, 2>);
+            if (vdim <= 4096) return row(zero, ns_gated_norm_row_kernel<T, 4>);
+            return row(zero, ns_gated_norm_row_kernel<T, 8>);
+        };
+        return out_dtype == NS_F32 ? pick(float(0)) : pick(uint16_t(0));
+    }
     const int64_t blocks = (rows * heads + 7) / 8, most = (int64_t)d->sm_count * 32;
     const dim3 grid((unsigned)(blocks < most ? blocks : most));
     if (out_dtype == NS_F32) {

@@ -125,12 +125,106 @@ __global__ void __launch_bounds__(256) ns_rms_rows_kernel(const RmsArgs a)
 }
 
 // ---------------------------------------------------------------------------------------------
-// y = gelu(source[:, 0:ff]) * source[:, ff:2ff]
+// x_out = x + source / sqrt(mean(source^2) + eps) * post_w (+ plus);  y = x_out / sqrt(mean(x_out^2) + eps) * w
 // ---------------------------------------------------------------------------------------------
-template <typename T>
-NS_DEVINL float glu_act(float g) { return sizeof(T) == 2 ? ns_gelu_fast(g) : ns_gelu_tanh(g); }
+struct PostRmsArgs {
+    RmsArgs r;               // alpha and row_map are not used
+    const float* post_w;
+    const float* plus;       // [rows, cols] or null
+};
 
-template <typename T, bool VEC>
+// Q: groups of four columns a thread keeps in registers
+template <typename T, int Q>
+__global__ void __launch_bounds__(256) ns_rms_post_rows_vec_kernel(const PostRmsArgs p)
+{
+    const RmsArgs& a = p.r;
+    __shared__ float red[2][8];
+    ns_pdl_wait();
+    ns_pdl_trigger();
+    const int row = blockIdx.x;
+    const int64_t base = (int64_t)row * a.cols;
+    float4 s[Q], x[Q];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int c = (threadIdx.x + 256 * i) * 4;
+        s[i] = x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= a.cols) continue;
+        s[i] = ns_source_at4(a.src, (int64_t)row * a.src.ld + c);
+        x[i] = *reinterpret_cast<const float4*>(a.x + base + c);
+        if (p.plus != nullptr) {
+            const float4 t = *reinterpret_cast<const float4*>(p.plus + base + c);
+            x[i] = make_float4(x[i].x + t.x, x[i].y + t.y, x[i].z + t.z, x[i].w + t.w);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < Q; i++) { ss = fmaf(s[i].x, s[i].x, ss); ss = fmaf(s[i].y, s[i].y, ss); ss = fmaf(s[i].z, s[i].z, ss); ss = fmaf(s[i].w, s[i].w, ss); }
+    const float post = 1.0f / sqrtf(ns_cta_sum(ss, red[0]) / (float)a.cols + a.eps);
+    ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int c = (threadIdx.x + 256 * i) * 4;
+        if (c >= a.cols) continue;
+        const float4 w = __ldg(reinterpret_cast<const float4*>(p.post_w + c));
+        x[i] = make_float4(fmaf(s[i].x * post, w.x, x[i].x), fmaf(s[i].y * post, w.y, x[i].y), fmaf(s[i].z * post, w.z, x[i].z), fmaf(s[i].w * post, w.w, x[i].w));
+        *reinterpret_cast<float4*>(a.x_out + base + c) = x[i];
+        ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss);
+    }
+    if (a.w == nullptr) return;
+    const float inv = 1.0f / sqrtf(ns_cta_sum(ss, red[1]) / (float)a.cols + a.eps);
+    T* y = reinterpret_cast<T*>(a.y) + (int64_t)row * a.y_ld;
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int c = (threadIdx.x + 256 * i) * 4;
+        if (c >= a.cols) continue;
+        const float4 w = __ldg(reinterpret_cast<const float4*>(a.w + c));
+        ns_store4(y + c, make_float4(x[i].x * inv * w.x, x[i].y * inv * w.y, x[i].z * inv * w.z, x[i].w * inv * w.w));
+    }
+    for (int c = a.cols + threadIdx.x; c < a.y_ld; c += blockDim.x) ns_store(y + c, 0.0f);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) ns_rms_post_rows_kernel(const PostRmsArgs p)
+{
+    const RmsArgs& a = p.r;
+    extern __shared__ float4 rms_row4[];
+    float* buf = reinterpret_cast<float*>(rms_row4);
+    __shared__ float red[2][8];
+    ns_pdl_wait();
+    ns_pdl_trigger();
+    const int row = blockIdx.x;
+    const int64_t base = (int64_t)row * a.cols;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < a.cols; c += blockDim.x) {
+        buf[c] = ns_source_at(a.src, (int64_t)row * a.src.ld + c);
+        ss = fmaf(buf[c], buf[c], ss);
+    }
+    const float post = 1.0f / sqrtf(ns_cta_sum(ss, red[0]) / (float)a.cols + a.eps);
+    ss = 0.0f;
+    for (int c = threadIdx.x; c < a.cols; c += blockDim.x) {
+        const float v = fmaf(buf[c] * post, p.post_w[c], a.x[base + c] + (p.plus != nullptr ? p.plus[base + c] : 0.0f));
+        a.x_out[base + c] = v;
+        ss = fmaf(v, v, ss);
+        buf[c] = v;
+    }
+    if (a.w == nullptr) return;
+    const float inv = 1.0f / sqrtf(ns_cta_sum(ss, red[1]) / (float)a.cols + a.eps);
+    T* y = reinterpret_cast<T*>(a.y) + (int64_t)row * a.y_ld;
+    for (int c = threadIdx.x; c < a.cols; c += blockDim.x) ns_store(y + c, buf[c] * inv * a.w[c]);
+    for (int c = a.cols + threadIdx.x; c < a.y_ld; c += blockDim.x) ns_store(y + c, 0.0f);
+}
+
+// ---------------------------------------------------------------------------------------------
+// y = act(source[:, 0:ff]) * source[:, ff:2ff]
+// ---------------------------------------------------------------------------------------------
+template <typename T, int ACT>
+NS_DEVINL float glu_act(float g)
+{
+    if (ACT == NS_ACT_RELU) return fmaxf(g, 0.0f);
+    return sizeof(T) == 2 ? ns_gelu_fast(g) : ns_gelu_tanh(g);
+}
+
+template <typename T, bool VEC, int ACT>
 __global__ void __launch_bounds__(256) ns_glu_rows_kernel(const NsSource s, int64_t rows, int ff, T* __restrict__ y, int64_t y_ld)
 {
     ns_pdl_wait();
@@ -144,7 +238,7 @@ __global__ void __launch_bounds__(256) ns_glu_rows_kernel(const NsSource s, int6
             float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
             if (c < ff) {
                 const float4 g = ns_source_at4(s, r * s.ld + c), u = ns_source_at4(s, r * s.ld + ff + c);
-                o = make_float4(glu_act<T>(g.x) * u.x, glu_act<T>(g.y) * u.y, glu_act<T>(g.z) * u.z, glu_act<T>(g.w) * u.w);
+                o = make_float4(glu_act<T, ACT>(g.x) * u.x, glu_act<T, ACT>(g.y) * u.y, glu_act<T, ACT>(g.z) * u.z, glu_act<T, ACT>(g.w) * u.w);
             }
             ns_store4(y + r * y_ld + c, o);
         }
@@ -154,7 +248,7 @@ __global__ void __launch_bounds__(256) ns_glu_rows_kernel(const NsSource s, int6
             const int64_t r = q / y_ld;
             const int c = (int)(q - r * y_ld);
             float o = 0.0f;
-            if (c < ff) o = glu_act<T>(ns_source_at(s, r * s.ld + c)) * ns_source_at(s, r * s.ld + ff + c);
+            if (c < ff) o = glu_act<T, ACT>(ns_source_at(s, r * s.ld + c)) * ns_source_at(s, r * s.ld + ff + c);
             ns_store(y + q, o);
         }
     }
@@ -262,22 +356,66 @@ extern "C" int ns_rms_rows(ns_device_t h, uint64_t x, uint64_t src, int splits, 
     return vec ? launch(ns_rms_rows_kernel<uint16_t, true>) : launch(ns_rms_rows_kernel<uint16_t, false>);
 }
 
-extern "C" int ns_glu_rows(ns_device_t h, uint64_t src, int splits, int src_dtype, int src_ld, int64_t rows, int ff, int out_dtype, uint64_t y, int y_ld)
+extern "C" int ns_rms_post_rows(ns_device_t h, uint64_t x, uint64_t src, int splits, int src_dtype, int src_ld, uint64_t post_w, uint64_t plus, uint64_t x_out, uint64_t w,
+                                float eps, int64_t rows, int cols, int out_dtype, uint64_t y, int y_ld)
 {
     NS_ENTER(h);
+    NS_REQUIRE(rows > 0 && cols > 0 && x && x_out && post_w, NS_ERR_ARGUMENT, "ns_rms_post_rows: bad argument");
+    NS_REQUIRE(ns_source_ok(src, splits, src_dtype) && src_ld >= cols, NS_ERR_ARGUMENT, "ns_rms_post_rows: bad source");
+    NS_REQUIRE(w == 0 || (y && float_or_bf16(out_dtype) && y_ld >= cols), NS_ERR_ARGUMENT, "ns_rms_post_rows: bad output");
+    NS_REQUIRE((size_t)cols * 4 <= 160 * 1024, NS_ERR_ARGUMENT, "ns_rms_post_rows: %d columns do not fit shared memory", cols);
+    PostRmsArgs p;
+    RmsArgs& a = p.r;
+    a.x = reinterpret_cast<const float*>(x);
+    a.src = ns_source(src, splits, src_dtype, rows, src_ld);
+    a.alpha = 1.0f;
+    a.x_out = reinterpret_cast<float*>(x_out);
+    a.w = reinterpret_cast<const float*>(w);
+    a.eps = eps;
+    a.row_map = nullptr;
+    a.cols = cols;
+    a.y = reinterpret_cast<void*>(y);
+    a.y_ld = y_ld;
+    p.post_w = reinterpret_cast<const float*>(post_w);
+    p.plus = reinterpret_cast<const float*>(plus);
+    const bool vec = ((cols | src_ld | (w ? y_ld : 0)) & 3) == 0 && ((x | src | x_out | w | y | post_w | plus) & 15) == 0 && (a.src.slab & 3) == 0 && cols <= 8192;
+    const size_t smem = vec ? 0 : (size_t)((cols + 3) & ~3) * 4;
+    auto launch = [&](auto kernel) -> int {
+        if (smem > 48 * 1024) NS_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        NS_CUDA(ns_launch_plain(kernel, dim3((unsigned)rows), dim3(256), smem, d->stream, p));
+        return NS_OK;
+    };
+    auto pick = [&](auto zero) -> int {
+        using T = decltype(zero);
+        if (!vec) return launch(ns_rms_post_rows_kernel<T>);
+        if (cols <= 1024) return launch(ns_rms_post_rows_vec_kernel<T, 1>);
+        if (cols <= 2048) return launch(ns_rms_post_rows_vec_kernel<T, 2>);
+        if (cols <= 4096) return launch(ns_rms_post_rows_vec_kernel<T, 4>);
+        return launch(ns_rms_post_rows_vec_kernel<T, 8>);
+    };
+    return w == 0 || out_dtype == NS_F32 ? pick(float(0)) : pick(uint16_t(0));
+}
+
+extern "C" int ns_glu_rows(ns_device_t h, uint64_t src, int splits, int src_dtype, int src_ld, int64_t rows, int ff, int act, int out_dtype, uint64_t y, int y_ld)
+{
+    NS_ENTER(h);
+    NS_REQUIRE(act == NS_ACT_GELU || act == NS_ACT_RELU, NS_ERR_ARGUMENT, "ns_glu_rows: unknown activation %d", act);
     NS_REQUIRE(rows > 0 && ff > 0 && y && y_ld >= ff && float_or_bf16(out_dtype), NS_ERR_ARGUMENT, "ns_glu_rows: bad argument");
     NS_REQUIRE(ns_source_ok(src, splits, src_dtype) && src_ld >= 2 * ff, NS_ERR_ARGUMENT, "ns_glu_rows: bad source");
     const NsSource s = ns_source(src, splits, src_dtype, rows, src_ld);
     const bool vec = ((ff | src_ld | y_ld) & 3) == 0 && ((src | y) & 15) == 0;
     const unsigned grid = flat_grid(d, vec ? rows * (y_ld / 4) : rows * y_ld);
+    auto launch = [&](auto zero, auto kernel) -> int {
+        using T = decltype(zero);
+        NS_CUDA(ns_launch_plain(kernel, dim3(grid), dim3(256), 0, d->stream, s, rows, ff, reinterpret_cast<T*>(y), (int64_t)y_ld));
+        return NS_OK;
+    };
     if (out_dtype == NS_F32) {
-        auto k = vec ? ns_glu_rows_kernel<float, true> : ns_glu_rows_kernel<float, false>;
-        NS_CUDA(ns_launch_plain(k, dim3(grid), dim3(256), 0, d->stream, s, rows, ff, reinterpret_cast<float*>(y), (int64_t)y_ld));
-    } else {
-        auto k = vec ? ns_glu_rows_kernel<uint16_t, true> : ns_glu_rows_kernel<uint16_t, false>;
-        NS_CUDA(ns_launch_plain(k, dim3(grid), dim3(256), 0, d->stream, s, rows, ff, reinterpret_cast<uint16_t*>(y), (int64_t)y_ld));
+        if (act == NS_ACT_RELU) return vec ? launch(float(0), ns_glu_rows_kernel<float, true, NS_ACT_RELU>) : launch(float(0), ns_glu_rows_kernel<float, false, NS_ACT_RELU>);
+        return vec ? launch(float(0), ns_glu_rows_kernel<float, true, NS_ACT_GELU>) : launch(float(0), ns_glu_rows_kernel<float, false, NS_ACT_GELU>);
     }
-    return NS_OK;
+    if (act == NS_ACT_RELU) return vec ? launch(uint16_t(0), ns_glu_rows_kernel<uint16_t, true, NS_ACT_RELU>) : launch(uint16_t(0), ns_glu_rows_kernel<uint16_t, false, NS_ACT_RELU>);
+    return vec ? launch(uint16_t(0), ns_glu_rows_kernel<uint16_t, true, NS_ACT_GELU>) : launch(uint16_t(0), ns_glu_rows_kernel<uint16_t, false, NS_ACT_GELU>);
 }
 
 extern "C" int ns_copy_cols(ns_device_t h, uint64_t src, int splits, int src_dtype, int src_ld, int col, int64_t rows, int cols, int out_dtype, uint64_t y,

@@ -14,7 +14,7 @@ LIB_PATH = os.path.join(_HERE, "libns_b200.so")
 
 NS_F32, NS_BF16, NS_I8, NS_I32 = 0, 1, 2, 3
 EPI_NONE, EPI_BIAS, EPI_BIAS_GELU, EPI_BIAS_RESIDUAL = 0, 1, 2, 3
-ACT_SILU, ACT_SIGMOID = 0, 1
+ACT_SILU, ACT_SIGMOID, ACT_GELU, ACT_RELU = 0, 1, 2, 3
 SPLIT_NONE, SPLIT_COLUMN, SPLIT_ROW = 0, 1, 2
 
 u64, i64, i32, u32, f32, vp, cp = C.c_uint64, C.c_int64, C.c_int, C.c_uint32, C.c_float, C.c_void_p, C.c_char_p
@@ -93,7 +93,8 @@ SIGNATURES = {
     "ns_linear_create_bf16": [vp, i32, i32, vp, P(vp)],
     "ns_embed_ngram": [vp, u64, u64, i32, i32, f32, u64, i32, i32, i64, i64, u64, u64, i32, i32, i32, i32, u64],
     "ns_rms_rows": [vp, u64, u64, i32, i32, i32, f32, u64, u64, f32, u64, i64, i64, i32, i32, u64, i32],
-    "ns_glu_rows": [vp, u64, i32, i32, i32, i64, i32, i32, u64, i32],
+    "ns_rms_post_rows": [vp, u64, u64, i32, i32, i32, u64, u64, u64, u64, f32, i64, i32, i32, u64, i32],
+    "ns_glu_rows": [vp, u64, i32, i32, i32, i64, i32, i32, i32, u64, i32],
     "ns_copy_cols": [vp, u64, i32, i32, i32, i32, i64, i32, i32, u64, i32],
     "ns_seq_advance": [vp, u64, u64, i32, i32, u64, u64],
     "ns_ids_from_f32": [vp, u64, u64, i32],
@@ -101,6 +102,12 @@ SIGNATURES = {
     "ns_delta_recurrent": [vp, u64, i32, u64, i32, u64, i32, u64, i32, i32, i32, u64, i32, i32, i32, u64, u64, i32, u64, i64, u64, i32, i32, i32, i32, i32, i32, u64, i32],
     "ns_delta_chunked": [vp, u64, i32, u64, i32, u64, i32, u64, i32, i32, i32, u64, i32, i32, i32, u64, u64, i32, u64, i64, u64, i32, i32, i32, i32, i32, i32, u64, i32],
     "ns_gated_norm": [vp, u64, i32, u64, i32, i32, i32, i32, i32, u64, f32, i64, i32, i32, i32, u64, i32],
+    "ns_lightning_recurrent": [vp, u64, i32, i32, i32, i32, i32, i32, u64, u64, u64, i64, u64, i32, i32, i32, i32, i32, u64, i32],
+    "ns_lightning_chunked": [vp, u64, i32, i32, i32, i32, i32, i32, u64, u64, u64, i64, u64, i32, i32, i32, i32, i32, u64, i32, i32],
+    "ns_window_append": [vp, u64, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, u64, u64, f32, u64, u64, i32, i32, i32, u64, u64, u64, u64, i64, i64, i32, i32, i32],
+    "ns_window_attend": [vp, i32, u64, u64, u64, i64, i64, i32, i32, i32, u64, u64, u64, u64, i32, i32, i32, i32, i32, i32, i32, f32, u64, i64],
+    "ns_window_decode": [vp, u64, u64, u64, i64, i64, i32, i32, i32, u64, u64, u64, u64, i32, i32, i32, i32, i32, i32, i32, f32, u64, i64],
+    "ns_window_prefill": [vp, u64, u64, u64, i64, i64, i32, i32, i32, i32, u64, u64, u64, u64, i32, i32, i32, i32, i32, i32, i32, f32, u64, i64],
     "ns_latent_append": [vp, u64, i32, i32, i32, i32, i32, i32, i32, u64, u64, f32, u64, u64, u64, i32, i32, i32, u64, i32, u64, i64, i32, i32],
     "ns_rotate_heads": [vp, u64, i32, i32, i32, i32, i32, i32, i32, u64, u64, u64, i32, i32, i32, u64, i64, i32, i32, u64, i64, i32],
     "ns_head_matmul": [vp, i32, u64, i64, i32, i32, u64, i64, i64, i64, i32, u64, i64, i32, i32, i32, i32, i32],

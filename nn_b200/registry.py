@@ -14,17 +14,30 @@ from .device import Device
 DTYPES = {"bfloat16": N.NS_BF16, "float32": N.NS_F32}
 
 
-def _fabezen(dev: Device, folder: str, config: dict, dtype: str, batch: int, max_prefill: int, slots: int | None):
+def _fabezen():
     from .fabezen import Fabezen, FabezenConfig
+
+    return Fabezen, FabezenConfig
+
+
+def _topidra():
+    from .topidra import Topidra, TopidraConfig
+
+    return Topidra, TopidraConfig
+
+
+# name -> () -> (decoder class, configuration class)
+ARCHITECTURES = {"Fabezen": _fabezen, "Topidra": _topidra}
+
+
+def _load_folder(dev: Device, folder: str, config: dict, dtype: str, batch: int, max_prefill: int, slots: int | None):
     from .weights import SafeTensors, check_shapes
 
-    cfg = FabezenConfig.from_dict(config)
+    model_class, config_class = ARCHITECTURES[config["architecture"]]()
+    cfg = config_class.from_dict(config)
     tensors = SafeTensors(os.path.join(folder, "model.safetensors"))
     check_shapes(tensors, cfg.tensor_shapes())
-    return Fabezen(dev, cfg, tensors, batch=batch, max_prefill=max_prefill, dtype=DTYPES[dtype], slots=slots)
-
-
-ARCHITECTURES = {"Fabezen": _fabezen}
+    return model_class(dev, cfg, tensors, batch=batch, max_prefill=max_prefill, dtype=DTYPES[dtype], slots=slots)
 
 
 def read_config(folder: str) -> dict:
@@ -42,7 +55,7 @@ def load_model(dev: Device, path: str, dtype: str = "bfloat16", batch: int = 1, 
         name = config.get("architecture")
         if name not in ARCHITECTURES:
             raise ValueError(f"{path}: architecture {name!r} is none of {', '.join(sorted(ARCHITECTURES))}")
-        return ARCHITECTURES[name](dev, path, config, dtype, batch, max_prefill, slots)
+        return _load_folder(dev, path, config, dtype, batch, max_prefill, slots)
     from .gpt import GptW8A8
     from .gpt_f32 import GptF32
     from .weights import load_char_gpt

@@ -118,7 +118,7 @@ def test_gated_linear_unit(dev, rows, ff, splits, out):
     s, ld = split_source(dev, x, splits, (2 * ff + 7) // 8 * 8)
     y_ld = (ff + 7) // 8 * 8
     y = dev.from_numpy(np.full(rows * y_ld, 9, np.float32 if out == N.NS_F32 else np.uint16))
-    N.call("ns_glu_rows", dev.handle, u(s.ptr), splits, N.NS_F32, ld, i64(rows), ff, out, u(y.ptr), y_ld)
+    N.call("ns_glu_rows", dev.handle, u(s.ptr), splits, N.NS_F32, ld, i64(rows), ff, N.ACT_GELU, out, u(y.ptr), y_ld)
     dev.synchronize()
     got = y.download((rows, y_ld)) if out == N.NS_F32 else f32(y.download((rows, y_ld)))
     close(got[:, :ff], F.gelu_tanh(x[:, :ff]) * x[:, ff:], 3e-6 if out == N.NS_F32 else 5e-2)
