@@ -840,8 +840,8 @@ def run_case(spec: str):
         print(json.dumps({"case": spec, "ok": True, "rows": m, "layer_us": total, "hbm_peak_gbs": peaks["hbm"], "ops": rows}))
         model.close()
         return
-    elif name == "fabezen":
-        print(json.dumps({"case": spec, "ok": True, **run_fabezen(dev, arg)}))
+    elif name in BLOCK_MODELS:
+        print(json.dumps({"case": spec, "ok": True, **run_block_model(dev, name, arg)}))
         return
     elif name == "gpt_decode":
         from nn_b200 import dist as nsdist
@@ -860,7 +860,7 @@ def run_case(spec: str):
 
 
 # ---------------------------------------------------------------------------------------------------------------
-# Fabezen beside the int8 decoder at equal size
+# the decoders made of blocks beside the int8 decoder at equal size
 # ---------------------------------------------------------------------------------------------------------------
 def fabezen_config(width: int, heads: int, ff: int, window: int, kinds: str, vocab: int = 32000, kv_rank: int = 512) -> dict:
     """kinds: one letter per layer, d(elta), c(hannel-wise delta), l(atent attention); a kind's later layers use its first one's
@@ -881,13 +881,26 @@ def fabezen_config(width: int, heads: int, ff: int, window: int, kinds: str, voc
             "embedding": {"scale": 8.0, "bigram": {"buckets": 32768, "mul_prev": 1009, "mul_cur": 31}}}
 
 
-class SyntheticFabezenWeights(dict):
+def topidra_config(width: int, heads: int, ff: int, window: int, kinds: str, vocab: int = 32000) -> dict:
+    """kinds: one letter per layer, a(ttention, as many key/value heads as heads), g(rouped: a quarter of them), l(ightning)."""
+    dim = width // heads
+    layers = []
+    for k in kinds:
+        if k == "l":
+            layers.append({"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** (-2 - 8 * i / heads) for i in range(heads)]}})
+        else:
+            layers.append({"type": "attention", "mixer": {"heads": heads, "kv_heads": {"a": heads, "g": heads // 4}[k], "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                          "mask": {"size": window}}})
+        layers[-1]["mlp"] = {"kind": "dense", "ff": ff}
+    return {"architecture": "Topidra", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-5}}
+
+
+class SyntheticBlockWeights(dict):
     """Random bf16 tensors made on first use; low ranks are the head size."""
 
-    def __init__(self, cfg: dict, low_rank: int):
-        from nn_b200.fabezen import FabezenConfig
+    def __init__(self, shapes: dict, low_rank: int):
         super().__init__()
-        self.shapes = {k: tuple(low_rank if n is None else n for n in s) for k, s in FabezenConfig.from_dict(cfg).tensor_shapes().items()}
+        self.shapes = {k: tuple(low_rank if n is None else n for n in s) for k, s in shapes.items()}
 
     def __getitem__(self, key: str):
         from nn_b200.blocks import bf16_bits
@@ -898,7 +911,7 @@ class SyntheticFabezenWeights(dict):
             x = 1.0 + 0.1 * x
         elif last in ("A_log", "dt_bias"):
             x -= 2.0
-        elif key != "embed" and key != "bigram":
+        elif key not in ("embed", "bigram") and last != "sink":
             x *= shape[-1] ** -0.5
         return bf16_bits(x)
 
@@ -917,6 +930,24 @@ def fabezen_step_bytes(model, batch: int, context: int) -> float:
         else:
             qk, v = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
             total += 2.0 * D * (2 * qk + 2 * v + v) + 8.0 * batch * m["heads"] * m["dim"] * m["vdim"]
+        if layer.mlp:
+            total += 6.0 * D * layer.mlp["ff"]
+    return total
+
+
+def topidra_step_bytes(model, batch: int, context: int) -> float:
+    """The same for Topidra; a layer's weights count once a run."""
+    cfg = model.cfg
+    D, total = cfg.width, 2.0 * cfg.vocab * cfg.width
+    for i, _ in cfg.runs():
+        layer = cfg.layers[i]
+        m = layer.mixer
+        H = m["heads"]
+        if layer.type == "attention":
+            kv = m["kv_heads"] * (m["dim"] + m["vdim"])
+            total += 2.0 * D * (H * m["dim"] + kv + H + H * m["vdim"]) + 2.0 * batch * min(context, m["mask"]["size"]) * kv
+        else:
+            total += 2.0 * D * H * (2 * m["dim"] + 3 * m["vdim"]) + 8.0 * batch * H * m["dim"] * m["vdim"]
         if layer.mlp:
             total += 6.0 * D * layer.mlp["ff"]
     return total
@@ -951,18 +982,25 @@ def time_calls(dev, run, reps: int = 10, skip=("ns_h2d",)):
     return out
 
 
-def run_fabezen(dev, arg: str) -> dict:
-    """fabezen[:width:heads:ff:window:kinds:batch:prompt:new[:parts]] -- prefill and decoding throughput with random weights, and the
+# design -> (configuration, algorithmic bytes of a decoding step, default layers)
+BLOCK_MODELS = {"fabezen": (fabezen_config, fabezen_step_bytes, "dcl"), "topidra": (topidra_config, topidra_step_bytes, "lal")}
+
+
+def run_block_model(dev, design: str, arg: str) -> dict:
+    """design[:width:heads:ff:window:kinds:batch:prompt:new[:parts]] -- prefill and decoding throughput with random weights, and the
     int8 decoder of equal width, heads, layers, batch and prompt beside it (its feed-forward has two matrices of 1.5 ff, as many
     weights as the gated one's three).  `parts` instead times every library call of one prompt read and one step."""
-    from nn_b200.fabezen import Fabezen, FabezenConfig
     from nn_b200.gpt import GptConfig, GptW8A8
+    from nn_b200.registry import ARCHITECTURES
+    config_of, step_bytes, default_kinds = BLOCK_MODELS[design]
     f = (arg.split(":") if arg else []) + [""] * 9
     width, heads, ff, window = int(f[0] or 2048), int(f[1] or 16), int(f[2] or 5632), int(f[3] or 512)
-    kinds, B, P, new = f[4] or "dcl", int(f[5] or 64), int(f[6] or 512), int(f[7] or 64)
+    kinds, B, P, new = f[4] or default_kinds, int(f[5] or 64), int(f[6] or 512), int(f[7] or 64)
     peaks = measured_peaks()
-    cfg = fabezen_config(width, heads, ff, window, kinds)
-    model = Fabezen(dev, FabezenConfig.from_dict(cfg), SyntheticFabezenWeights(cfg, width // heads), batch=B, max_prefill=P)
+    cfg = config_of(width, heads, ff, window, kinds)
+    model_class, config_class = ARCHITECTURES[cfg["architecture"]]()
+    mcfg = config_class.from_dict(cfg)
+    model = model_class(dev, mcfg, SyntheticBlockWeights(mcfg.tensor_shapes(), width // heads), batch=B, max_prefill=P)
     prompt = np.random.default_rng(5).integers(0, cfg["vocab"], (B, P)).astype(np.int32)
     if f[8] == "parts":
         model.generate(prompt, 4)
@@ -977,7 +1015,7 @@ def run_fabezen(dev, arg: str) -> dict:
 
     def timed(m):
         m.generate(prompt, min(new, 8))
-        sampler = ClockSampler(dev.ordinal, "_fabezen")
+        sampler = ClockSampler(dev.ordinal, "_" + design)
         sampler.start()
         marks = {}
         m.generate(prompt, new, marks=marks)
@@ -986,7 +1024,7 @@ def run_fabezen(dev, arg: str) -> dict:
                 "launches_per_step": m.launches_per_step, "clocks": clocks}
 
     rec = timed(model)
-    bytes_ = fabezen_step_bytes(model, B, P + new // 2)
+    bytes_ = step_bytes(model, B, P + new // 2)
     model.close()
     ctx = P + new
     gcfg = GptConfig(vocab=cfg["vocab"], dim=width, heads=heads, layers=len(kinds), ff_dim=3 * ff // 2 // 256 * 256, context=ctx)
@@ -999,7 +1037,7 @@ def run_fabezen(dev, arg: str) -> dict:
         r["decode_tokens_per_s"] = B / (r["ms_per_step"] * 1e-3)
         r["decode_hbm_frac"] = nbytes / (r["ms_per_step"] * 1e-3) / 1e9 / peaks["hbm"]
     return {"config": {"width": width, "heads": heads, "ff": ff, "window": window, "layers": kinds, "batch": B, "prompt": P, "new_tokens": new,
-                       "weights": "random, bf16", "peaks": peaks["source"]}, "fabezen": rec, "int8_gpt_equal_size": ref}
+                       "weights": "random, bf16", "peaks": peaks["source"]}, design: rec, "int8_gpt_equal_size": ref}
 
 
 def main():

@@ -67,7 +67,6 @@ __global__ void __launch_bounds__(256) ns_lightning_recurrent_kernel(const Light
         }
         if (tid < VT) sv[s][tid] = v0 + tid < vdim ? ns_silu(pv) : 0.0f;
     };
-    fetch(0);
     float st[RPW][V];
 #pragma unroll
     for (int i = 0; i < RPW; i++) {
@@ -88,6 +87,7 @@ __global__ void __launch_bounds__(256) ns_lightning_recurrent_kernel(const Light
                 if (col + j < vdim) st[i][j] = p[j];
         }
     }
+    fetch(0);
     put(0);
     __syncthreads();
     for (int t = 0; t < a.steps; t++) {
@@ -139,13 +139,20 @@ __global__ void __launch_bounds__(256) ns_lightning_recurrent_kernel(const Light
 // chunks of 64 tokens
 // ---------------------------------------------------------------------------------------------
 constexpr int LC = 64;        // tokens per chunk
-constexpr int LDV = 64;       // value columns per CTA
 
-template <int DK>
-struct LightningSmem {
-    static constexpr int LK = DK + 8, LV = LDV + 8;                   // row lengths that keep ldmatrix free of bank conflicts
-    static constexpr int Q = 0, K = Q + LC * LK * 2, V = K + LC * LK * 2, VH = V + LC * LV * 2, VL = VH + LC * LV * 2, SH = VL + LC * LV * 2,
-                         SL = SH + DK * LV * 2, TOTAL = SL + DK * LV * 2;
+// A CTA handles up to DV value columns with DV * 4 threads: 16 rows x 32 columns of a chunk's outputs per warp.
+template <int DK, int DV>
+struct LightningShape {
+    static constexpr int THREADS = DV * 4, WARPS = DV / 8;
+    // rows that keep ldmatrix free of bank conflicts, in elements
+    static constexpr int LK = DK + 8, LV = DV + 8, LP = LC + 8;
+    // shared memory: queries, keys, values (two chunks), values as the chunk's end sees them, the state, weighted scores (two chunks); the
+    // last three as two halves each
+    static constexpr int K_BYTES = LC * LK * 2, V_BYTES = LC * LV * 2, S_BYTES = DK * LV * 2, P_BYTES = LC * LP * 2;
+    static constexpr int Q = 0, K = Q + K_BYTES, V = K + K_BYTES, W = V + 2 * V_BYTES, S = W + 2 * V_BYTES, P = S + 2 * S_BYTES, TOTAL = P + 4 * P_BYTES;
+    // state tile of a warp: MT x 16 rows, NT x 8 columns
+    static constexpr int MT = DK >= 128 ? 2 : 1, ROW_GROUPS = DK / (16 * MT), NT = DV / 8 / (WARPS / ROW_GROUPS);
+    static_assert(TOTAL <= 227 * 1024 && NT % 2 == 0, "a CTA's shared memory");
 };
 
 // the bf16 halves of two values: x = hi + lo up to 2^-17 of x
@@ -157,48 +164,96 @@ NS_DEVINL void halves(float x, float y, uint32_t& hi, uint32_t& lo)
 NS_DEVINL void st_shared_v2(uint32_t addr, uint32_t a, uint32_t b) { asm volatile("st.shared.v2.b32 [%0], {%1, %2};" ::"r"(addr), "r"(a), "r"(b) : "memory"); }
 NS_DEVINL void st_shared_1(uint32_t addr, uint32_t a) { asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(a) : "memory"); }
 // z / (1 + e^-z); what it makes is rounded to bf16
-NS_DEVINL float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
-
-// Up to N groups of four neighbouring channels of the tile [64, width] at column `col` of a row, activated, as bf16 pairs.  Group x of a
-// thread is element tid + 256 x.  Rows past n and channels past size are zero.
-template <int WIDTH, int N>
-NS_DEVINL void load_silu(const NsSource& s, int64_t row0, int n, int col, int first, int size, bool vec, int tid, uint2 (&out)[N])
+NS_DEVINL float silu_fast(float z)
 {
-    constexpr int QUADS = WIDTH / 4;
-    float4 x[N];
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + ns_exp2(z * -1.4426950408889634f)));
+    return z * r;
+}
+
+// A tile [64, WIDTH] of the source from column `col` on, activated, as bf16 pairs: groups of four neighbouring channels, or of eight where the
+// source is one bf16 matrix (BF16).  Group x of a thread is element tid + THREADS x.  Rows past n and channels from `size` on are zero.
+// All loads are on their way before the first is used.
+template <int WIDTH, int THREADS, bool BF16>
+struct Tile {
+    static constexpr int PER = BF16 ? 8 : 4, GROUPS = WIDTH / PER, N = LC * GROUPS / THREADS > 0 ? LC * GROUPS / THREADS : 1;
+    uint32_t x[N][PER / 2];
+
+    NS_DEVINL static int row(int i, int tid) { return (tid + THREADS * i) / GROUPS; }
+    NS_DEVINL static int column(int i, int tid) { return (tid + THREADS * i) % GROUPS * PER; }
+
+    NS_DEVINL void load(const NsSource& s, int64_t row0, int n, int col, int size, bool vec, int tid)
+    {
+        if constexpr (BF16) {
+            const uint16_t* p = reinterpret_cast<const uint16_t*>(s.ptr) + row0 * s.ld + col;
 #pragma unroll
-    for (int i = 0; i < N; i++) {
-        const int e = tid + 256 * i, t = e / QUADS, c = first + (e % QUADS) * 4;
-        x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (t < n && c < size) {
-            const int64_t at = (row0 + t) * s.ld + col + c;
-            if (vec) {
-                x[i] = ns_source_at4(s, at);
-            } else {
-                x[i].x = ns_source_at(s, at);
-                if (c + 1 < size) x[i].y = ns_source_at(s, at + 1);
-                if (c + 2 < size) x[i].z = ns_source_at(s, at + 2);
-                if (c + 3 < size) x[i].w = ns_source_at(s, at + 3);
+            for (int i = 0; i < N; i++) {
+                const int t = row(i, tid), c = column(i, tid);
+                uint4 v = make_uint4(0, 0, 0, 0);
+                if (t < n && t < LC && c < size) v = *reinterpret_cast<const uint4*>(p + (int64_t)t * s.ld + c);
+                x[i][0] = v.x; x[i][1] = v.y; x[i][2] = v.z; x[i][3] = v.w;
+            }
+        } else {
+            float4 f[N];
+#pragma unroll
+            for (int i = 0; i < N; i++) {
+                const int t = row(i, tid), c = column(i, tid);
+                f[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (t >= n || t >= LC || c >= size) continue;
+                const int64_t at = (row0 + t) * s.ld + col + c;
+                if (vec) {
+                    f[i] = ns_source_at4(s, at);
+                } else {
+                    f[i].x = ns_source_at(s, at);
+                    if (c + 1 < size) f[i].y = ns_source_at(s, at + 1);
+                    if (c + 2 < size) f[i].z = ns_source_at(s, at + 2);
+                    if (c + 3 < size) f[i].w = ns_source_at(s, at + 3);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < N; i++) {
+                x[i][0] = ns_pack_bf16x2(silu_fast(f[i].x), silu_fast(f[i].y));
+                x[i][1] = ns_pack_bf16x2(silu_fast(f[i].z), silu_fast(f[i].w));
             }
         }
     }
+    NS_DEVINL void activate()
+    {
+        if constexpr (BF16) {
 #pragma unroll
-    for (int i = 0; i < N; i++)
-        out[i] = make_uint2(ns_pack_bf16x2(silu_fast(x[i].x), silu_fast(x[i].y)), ns_pack_bf16x2(silu_fast(x[i].z), silu_fast(x[i].w)));
-}
+            for (int i = 0; i < N; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) x[i][j] = ns_pack_bf16x2(silu_fast(__uint_as_float(x[i][j] << 16)), silu_fast(__uint_as_float(x[i][j] & 0xFFFF0000u)));
+        }
+    }
+    NS_DEVINL void store(uint32_t dst, int ld, int tid) const
+    {
+#pragma unroll
+        for (int i = 0; i < N; i++) {
+            if (row(i, tid) >= LC) continue;
+            const uint32_t at = dst + (row(i, tid) * ld + column(i, tid)) * 2;
+            if constexpr (BF16) ns_st_shared_v4(at, x[i][0], x[i][1], x[i][2], x[i][3]);
+            else st_shared_v2(at, x[i][0], x[i][1]);
+        }
+    }
+};
 
-// WRITES_ONLY: a segment's own writes (no queries, no outputs), left in seg_state.
-template <int DK, bool WRITES_ONLY>
-__global__ void __launch_bounds__(256, 2) ns_lightning_chunk_kernel(const LightningArgs a, int vec)
+// WRITES_ONLY: a segment's own writes (no queries, no outputs), left in seg_state.  BF16: the source is one bf16 matrix and every
+// tensor's columns start and end on multiples of eight; the next chunk's rows are then on their way while this one is computed.
+//
+// Between the first barrier of a chunk (its tiles and the state are in shared memory) and the second one, ten of the warps' 16 x 16
+// blocks of scores are made, weighted and left in shared memory, every warp reads the state out for its rows and takes the
+// chunk's writes into its piece of the state; after the second barrier the weighted scores meet the values.
+template <int DK, int DV, bool WRITES_ONLY, bool BF16>
+__global__ void __launch_bounds__(DV * 4, LightningShape<DK, DV>::TOTAL <= 113 * 1024 ? 2 : 1) ns_lightning_chunk_kernel(const LightningArgs a, int vec)
 {
-    using L = LightningSmem<DK>;
-    constexpr int ROW_TILES = DK / 16, COL_PARTS = 8 / ROW_TILES, NS = LDV / 8 / COL_PARTS;     // state tile of a warp: 16 rows, NS x 8 columns
+    using L = LightningShape<DK, DV>;
+    constexpr int MT = L::MT, NT = L::NT, T = L::THREADS;
     extern __shared__ __align__(16) uint8_t lc_smem[];
-    const uint32_t base = ns_smem_u32(lc_smem), sQ = base + L::Q, sK = base + L::K, sV = base + L::V, sVH = base + L::VH, sVL = base + L::VL,
-                   sSH = base + L::SH, sSL = base + L::SL;
+    const uint32_t base = ns_smem_u32(lc_smem), sQ = base + L::Q, sK = base + L::K, sWH = base + L::W, sWL = sWH + L::V_BYTES, sSH = base + L::S, sSL = sSH + L::S_BYTES;
     ns_pdl_wait();
     ns_pdl_trigger();
-    const int head = blockIdx.x, b = blockIdx.y, seg = blockIdx.z % a.segs, v0 = (blockIdx.z / a.segs) * LDV;
+    const int head = blockIdx.x, b = blockIdx.y, seg = blockIdx.z % a.segs, v0 = (blockIdx.z / a.segs) * DV;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const int dim = a.dim, vdim = a.vdim;
     const float ld2 = a.decay_log2[head];
@@ -206,86 +261,82 @@ __global__ void __launch_bounds__(256, 2) ns_lightning_chunk_kernel(const Lightn
     float* S = a.segs > 1 ? a.seg_state + (((int64_t)b * a.segs + seg) * a.heads + head) * per_head
                           : a.state + (int64_t)a.slots[b] * a.state_slot_stride + head * per_head;
     const int begin = seg * a.seg_len, end = min(a.steps, begin + a.seg_len);
-    const int sr = (warp % ROW_TILES) * 16, sc = (warp / ROW_TILES) * NS * 8;
+    const int sr = (warp % L::ROW_GROUPS) * MT * 16, sc = (warp / L::ROW_GROUPS) * NT * 8;
 
-    float st[NS][4];
-#pragma unroll
-    for (int j = 0; j < NS; j++)
-#pragma unroll
-        for (int e = 0; e < 4; e++) {
-            const int r = sr + g + (e >> 1) * 8, c = v0 + sc + j * 8 + t4 * 2 + (e & 1);
-            st[j][e] = !WRITES_ONLY && r < dim && c < vdim ? S[(int64_t)r * vdim + c] : 0.0f;
-        }
-
-    for (int c0 = begin; c0 < end; c0 += LC) {
+    Tile<DK, T, BF16> kt, qt;
+    Tile<DV, T, BF16> vt;
+    auto load_tiles = [&](int c0) {
         const int n = min(LC, end - c0);
         const int64_t row0 = (int64_t)b * a.steps + c0;
-        {
-            constexpr int NQ = LC * DK / 1024, NVG = LC * LDV / 1024;
-            uint2 kx[NQ], qx[WRITES_ONLY ? 1 : NQ], vx[NVG];
-            load_silu<DK, NQ>(a.src, row0, n, a.k_col + head * dim, 0, dim, vec, tid, kx);
-            if constexpr (!WRITES_ONLY) load_silu<DK, NQ>(a.src, row0, n, a.q_col + head * dim, 0, dim, vec, tid, qx);
-            load_silu<LDV, NVG>(a.src, row0, n, a.v_col + head * vdim, v0, vdim, vec, tid, vx);
+        kt.load(a.src, row0, n, a.k_col + head * dim, dim, vec, tid);
+        if constexpr (!WRITES_ONLY) qt.load(a.src, row0, n, a.q_col + head * dim, dim, vec, tid);
+        vt.load(a.src, row0, n, a.v_col + head * vdim + v0, vdim - v0, vec, tid);
+    };
+    load_tiles(begin);
+
+    float st[MT][NT][4];
 #pragma unroll
-            for (int i = 0; i < NQ; i++) {
-                const int e = tid + 256 * i, t = e / (DK / 4), c = (e % (DK / 4)) * 4;
-                st_shared_v2(sK + (t * L::LK + c) * 2, kx[i].x, kx[i].y);
-                if constexpr (!WRITES_ONLY) st_shared_v2(sQ + (t * L::LK + c) * 2, qx[i].x, qx[i].y);
+    for (int i = 0; i < MT; i++)
+#pragma unroll
+        for (int j = 0; j < NT; j++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int r = sr + i * 16 + g + (e >> 1) * 8, c = v0 + sc + j * 8 + t4 * 2 + (e & 1);
+                st[i][j][e] = !WRITES_ONLY && r < dim && c < vdim ? S[(int64_t)r * vdim + c] : 0.0f;
             }
+
+    for (int c0 = begin, turn = 0; c0 < end; c0 += LC, turn ^= 1) {
+        const int n = min(LC, end - c0);
+        const uint32_t sV = base + L::V + turn * L::V_BYTES, sPH = base + L::P + turn * 2 * L::P_BYTES, sPL = sPH + L::P_BYTES;
+        if (!BF16 && c0 > begin) load_tiles(c0);
+        kt.activate();
+        kt.store(sK, L::LK, tid);
+        if constexpr (!WRITES_ONLY) {
+            qt.activate();
+            qt.store(sQ, L::LK, tid);
+        }
+        vt.activate();
+        if constexpr (!WRITES_ONLY) vt.store(sV, L::LV, tid);
+        // the values as the state at the chunk's end sees them
+        using VT = Tile<DV, T, BF16>;
 #pragma unroll
-            for (int i = 0; i < NVG; i++) {
-                const int e = tid + 256 * i, t = e / (LDV / 4), c = (e % (LDV / 4)) * 4;
-                const uint32_t at = (t * L::LV + c) * 2;
-                if constexpr (!WRITES_ONLY) st_shared_v2(sV + at, vx[i].x, vx[i].y);
-                // the values as the state at the chunk's end sees them
-                const float w = t < n ? ns_exp2((float)(n - 1 - t) * ld2) : 0.0f;
-                uint32_t h0, l0, h1, l1;
-                halves(__uint_as_float(vx[i].x << 16) * w, __uint_as_float(vx[i].x & 0xFFFF0000u) * w, h0, l0);
-                halves(__uint_as_float(vx[i].y << 16) * w, __uint_as_float(vx[i].y & 0xFFFF0000u) * w, h1, l1);
-                st_shared_v2(sVH + at, h0, h1);
-                st_shared_v2(sVL + at, l0, l1);
+        for (int i = 0; i < VT::N; i++) {
+            const int t = VT::row(i, tid);
+            const float w = t < n ? ns_exp2((float)(n - 1 - t) * ld2) : 0.0f;
+            uint32_t hi[VT::PER / 2], lo[VT::PER / 2];
+#pragma unroll
+            for (int j = 0; j < VT::PER / 2; j++) halves(__uint_as_float(vt.x[i][j] << 16) * w, __uint_as_float(vt.x[i][j] & 0xFFFF0000u) * w, hi[j], lo[j]);
+            const uint32_t at = (t * L::LV + VT::column(i, tid)) * 2;
+            if constexpr (BF16) {
+                ns_st_shared_v4(sWH + at, hi[0], hi[1], hi[2], hi[3]);
+                ns_st_shared_v4(sWL + at, lo[0], lo[1], lo[2], lo[3]);
+            } else {
+                st_shared_v2(sWH + at, hi[0], hi[1]);
+                st_shared_v2(sWL + at, lo[0], lo[1]);
             }
-            if constexpr (!WRITES_ONLY) {
+        }
+        if constexpr (!WRITES_ONLY) {
 #pragma unroll
-                for (int j = 0; j < NS; j++)
+            for (int i = 0; i < MT; i++)
+#pragma unroll
+                for (int j = 0; j < NT; j++)
 #pragma unroll
                     for (int h = 0; h < 2; h++) {
                         uint32_t hi, lo;
-                        halves(st[j][2 * h], st[j][2 * h + 1], hi, lo);
-                        const uint32_t at = ((sr + g + h * 8) * L::LV + sc + j * 8 + t4 * 2) * 2;
+                        halves(st[i][j][2 * h], st[i][j][2 * h + 1], hi, lo);
+                        const uint32_t at = ((sr + i * 16 + g + h * 8) * L::LV + sc + j * 8 + t4 * 2) * 2;
                         st_shared_1(sSH + at, hi);
                         st_shared_1(sSL + at, lo);
                     }
-            }
         }
         __syncthreads();
+        if (BF16 && c0 + LC < end) load_tiles(c0 + LC);
+        const int r0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;       // this warp's outputs
+        float acc[4][4];
         if constexpr (!WRITES_ONLY) {
-            // 16 rows x 32 value columns per warp
-            const int r0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;
-            float acc[4][4];
-#pragma unroll
-            for (int j = 0; j < 4; j++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) acc[j][e] = 0.0f;
-            uint32_t qf[DK / 16][4];
-#pragma unroll
-            for (int k = 0; k < DK / 16; k++) {
-                ns_ldsm4(qf[k], ns_addr_a(sQ, L::LK, r0, k * 16, lane));
-                uint32_t bh[2][4], bl[2][4];
-#pragma unroll
-                for (int j = 0; j < 2; j++) {
-                    ns_ldsm4_t(bh[j], ns_addr_bt(sSH, L::LV, k * 16, n0 + j * 16, lane));
-                    ns_ldsm4_t(bl[j], ns_addr_bt(sSL, L::LV, k * 16, n0 + j * 16, lane));
-                }
-#pragma unroll
-                for (int j = 0; j < 4; j++) ns_mma_bf16(acc[j], qf[k], bh[j >> 1][2 * (j & 1)], bh[j >> 1][2 * (j & 1) + 1]);
-#pragma unroll
-                for (int j = 0; j < 4; j++) ns_mma_bf16(acc[j], qf[k], bl[j >> 1][2 * (j & 1)], bl[j >> 1][2 * (j & 1) + 1]);
-            }
-            const float f0 = ns_exp2((float)(r0 + g + 1) * ld2), f1 = ns_exp2((float)(r0 + g + 9) * ld2);
-#pragma unroll
-            for (int j = 0; j < 4; j++) { acc[j][0] *= f0; acc[j][1] *= f0; acc[j][2] *= f1; acc[j][3] *= f1; }
-            for (int kb = 0; kb <= r0; kb += 16) {
+            // blocks (0, 0), (1, 0), (1, 1), (2, 0), ... of the scores
+            for (int block = warp; block < 10; block += L::WARPS) {
+                const int qb = block < 1 ? 0 : (block < 3 ? 1 : (block < 6 ? 2 : 3)), kb = block - qb * (qb + 1) / 2;
                 float s[2][4];
 #pragma unroll
                 for (int j = 0; j < 2; j++)
@@ -293,24 +344,83 @@ __global__ void __launch_bounds__(256, 2) ns_lightning_chunk_kernel(const Lightn
                     for (int e = 0; e < 4; e++) s[j][e] = 0.0f;
 #pragma unroll
                 for (int k = 0; k < DK / 16; k++) {
-                    uint32_t bf[4];
-                    ns_ldsm4(bf, ns_addr_b(sK, L::LK, kb, k * 16, lane));
-                    ns_mma_bf16(s[0], qf[k], bf[0], bf[1]);
-                    ns_mma_bf16(s[1], qf[k], bf[2], bf[3]);
+                    uint32_t af[4], bf[4];
+                    ns_ldsm4(af, ns_addr_a(sQ, L::LK, qb * 16, k * 16, lane));
+                    ns_ldsm4(bf, ns_addr_b(sK, L::LK, kb * 16, k * 16, lane));
+                    ns_mma_bf16(s[0], af, bf[0], bf[1]);
+                    ns_mma_bf16(s[1], af, bf[2], bf[3]);
                 }
 #pragma unroll
                 for (int j = 0; j < 2; j++)
 #pragma unroll
-                    for (int e = 0; e < 4; e++) {
-                        const int back = r0 + g + (e >> 1) * 8 - (kb + j * 8 + t4 * 2 + (e & 1));
-                        s[j][e] = back >= 0 ? s[j][e] * ns_exp2((float)back * ld2) : 0.0f;
+                    for (int h = 0; h < 2; h++) {
+                        const int r = qb * 16 + g + h * 8, c = kb * 16 + j * 8 + t4 * 2;
+                        const float x = r >= c ? s[j][2 * h] * ns_exp2((float)(r - c) * ld2) : 0.0f;
+                        const float y = r >= c + 1 ? s[j][2 * h + 1] * ns_exp2((float)(r - c - 1) * ld2) : 0.0f;
+                        uint32_t hi, lo;
+                        halves(x, y, hi, lo);
+                        st_shared_1(sPH + (r * L::LP + c) * 2, hi);
+                        st_shared_1(sPL + (r * L::LP + c) * 2, lo);
                     }
-                uint32_t ph[4], pl[4];
-                halves(s[0][0], s[0][1], ph[0], pl[0]);
-                halves(s[0][2], s[0][3], ph[1], pl[1]);
-                halves(s[1][0], s[1][1], ph[2], pl[2]);
-                halves(s[1][2], s[1][3], ph[3], pl[3]);
-                uint32_t vf[2][4];
+            }
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[j][e] = 0.0f;
+#pragma unroll
+            for (int k = 0; k < DK / 16; k++) {
+                uint32_t af[4], bh[2][4], bl[2][4];
+                ns_ldsm4(af, ns_addr_a(sQ, L::LK, r0, k * 16, lane));
+#pragma unroll
+                for (int j = 0; j < 2; j++) {
+                    ns_ldsm4_t(bh[j], ns_addr_bt(sSH, L::LV, k * 16, n0 + j * 16, lane));
+                    ns_ldsm4_t(bl[j], ns_addr_bt(sSL, L::LV, k * 16, n0 + j * 16, lane));
+                }
+#pragma unroll
+                for (int j = 0; j < 4; j++) ns_mma_bf16(acc[j], af, bh[j >> 1][2 * (j & 1)], bh[j >> 1][2 * (j & 1) + 1]);
+#pragma unroll
+                for (int j = 0; j < 4; j++) ns_mma_bf16(acc[j], af, bl[j >> 1][2 * (j & 1)], bl[j >> 1][2 * (j & 1) + 1]);
+            }
+            const float f0 = ns_exp2((float)(r0 + g + 1) * ld2), f1 = ns_exp2((float)(r0 + g + 9) * ld2);
+#pragma unroll
+            for (int j = 0; j < 4; j++) { acc[j][0] *= f0; acc[j][1] *= f0; acc[j][2] *= f1; acc[j][3] *= f1; }
+        }
+        // the state after the chunk
+        const float fn = ns_exp2((float)n * ld2);
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int j = 0; j < NT; j++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) st[i][j][e] *= fn;
+#pragma unroll
+        for (int k = 0; k < LC; k += 16) {
+            uint32_t af[MT][4];
+#pragma unroll
+            for (int i = 0; i < MT; i++) ns_ldsm4_t(af[i], ns_addr_at(sK, L::LK, sr + i * 16, k, lane));
+#pragma unroll
+            for (int j = 0; j < NT; j += 2) {
+                uint32_t bh[4], bl[4];
+                ns_ldsm4_t(bh, ns_addr_bt(sWH, L::LV, k, sc + j * 8, lane));
+                ns_ldsm4_t(bl, ns_addr_bt(sWL, L::LV, k, sc + j * 8, lane));
+#pragma unroll
+                for (int i = 0; i < MT; i++) {
+                    ns_mma_bf16(st[i][j], af[i], bh[0], bh[1]);
+                    ns_mma_bf16(st[i][j + 1], af[i], bh[2], bh[3]);
+                }
+#pragma unroll
+                for (int i = 0; i < MT; i++) {
+                    ns_mma_bf16(st[i][j], af[i], bl[0], bl[1]);
+                    ns_mma_bf16(st[i][j + 1], af[i], bl[2], bl[3]);
+                }
+            }
+        }
+        __syncthreads();
+        if constexpr (!WRITES_ONLY) {
+            for (int kb = 0; kb <= r0; kb += 16) {
+                uint32_t ph[4], pl[4], vf[2][4];
+                ns_ldsm4(ph, ns_addr_a(sPH, L::LP, r0, kb, lane));
+                ns_ldsm4(pl, ns_addr_a(sPL, L::LP, r0, kb, lane));
 #pragma unroll
                 for (int j = 0; j < 2; j++) ns_ldsm4_t(vf[j], ns_addr_bt(sV, L::LV, kb, n0 + j * 16, lane));
 #pragma unroll
@@ -322,7 +432,7 @@ __global__ void __launch_bounds__(256, 2) ns_lightning_chunk_kernel(const Lightn
             for (int h = 0; h < 2; h++) {
                 const int r = r0 + g + h * 8;
                 if (r >= n) continue;
-                float* o = a.o + (row0 + r) * a.o_ld + (int64_t)head * vdim;
+                float* o = a.o + ((int64_t)b * a.steps + c0 + r) * a.o_ld + (int64_t)head * vdim;
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const int c = v0 + n0 + j * 8 + t4 * 2;
@@ -335,37 +445,17 @@ __global__ void __launch_bounds__(256, 2) ns_lightning_chunk_kernel(const Lightn
                 }
             }
         }
-        // the state after the chunk
-        const float fn = ns_exp2((float)n * ld2);
-#pragma unroll
-        for (int j = 0; j < NS; j++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) st[j][e] *= fn;
-#pragma unroll
-        for (int k = 0; k < LC; k += 16) {
-            uint32_t af[4];
-            ns_ldsm4_t(af, ns_addr_at(sK, L::LK, sr, k, lane));
-#pragma unroll
-            for (int j = 0; j < NS; j += 2) {
-                uint32_t bh[4], bl[4];
-                ns_ldsm4_t(bh, ns_addr_bt(sVH, L::LV, k, sc + j * 8, lane));
-                ns_ldsm4_t(bl, ns_addr_bt(sVL, L::LV, k, sc + j * 8, lane));
-                ns_mma_bf16(st[j], af, bh[0], bh[1]);
-                ns_mma_bf16(st[j + 1], af, bh[2], bh[3]);
-                ns_mma_bf16(st[j], af, bl[0], bl[1]);
-                ns_mma_bf16(st[j + 1], af, bl[2], bl[3]);
-            }
-        }
-        __syncthreads();
     }
     if (!WRITES_ONLY && a.segs > 1) return;          // the states at the segments' ends are known already
 #pragma unroll
-    for (int j = 0; j < NS; j++)
+    for (int i = 0; i < MT; i++)
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-            const int r = sr + g + (e >> 1) * 8, c = v0 + sc + j * 8 + t4 * 2 + (e & 1);
-            if (r < dim && c < vdim) S[(int64_t)r * vdim + c] = st[j][e];
-        }
+        for (int j = 0; j < NT; j++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int r = sr + i * 16 + g + (e >> 1) * 8, c = v0 + sc + j * 8 + t4 * 2 + (e & 1);
+                if (r < dim && c < vdim) S[(int64_t)r * vdim + c] = st[i][j][e];
+            }
 }
 
 // the segments' writes become the states before them; the state after the last goes to the slot
@@ -404,27 +494,34 @@ int launch_recurrent_rows(NsDevice* d, const LightningArgs& a, int batch)
     return launch_recurrent<32, V>(d, a, batch);
 }
 
-template <int DK, bool WRITES_ONLY>
+template <int DK, int DV, bool WRITES_ONLY, bool BF16>
 int launch_chunk_kernel(NsDevice* d, const LightningArgs& a, int batch, int vec)
 {
-    constexpr int smem = LightningSmem<DK>::TOTAL;
-    auto k = ns_lightning_chunk_kernel<DK, WRITES_ONLY>;
-    NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    const dim3 grid((unsigned)a.heads, (unsigned)batch, (unsigned)((a.vdim + LDV - 1) / LDV * a.segs));
-    NS_CUDA(ns_launch_plain(k, grid, dim3(256), (size_t)smem, d->stream, a, vec));
+    using L = LightningShape<DK, DV>;
+    auto k = ns_lightning_chunk_kernel<DK, DV, WRITES_ONLY, BF16>;
+    NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL));
+    const dim3 grid((unsigned)a.heads, (unsigned)batch, (unsigned)((a.vdim + DV - 1) / DV * a.segs));
+    NS_CUDA(ns_launch_plain(k, grid, dim3(L::THREADS), (size_t)L::TOTAL, d->stream, a, vec));
     return NS_OK;
 }
 
-template <int DK>
+template <int DK, int DV, bool BF16>
 int launch_chunked(NsDevice* d, const LightningArgs& a, int batch, int vec)
 {
     if (a.segs > 1) {
-        int rc = launch_chunk_kernel<DK, true>(d, a, batch, vec);
+        int rc = launch_chunk_kernel<DK, DV, true, BF16>(d, a, batch, vec);
         if (rc != NS_OK) return rc;
         const dim3 grid((unsigned)(((int64_t)a.dim * a.vdim + 255) / 256), (unsigned)a.heads, (unsigned)batch);
         NS_CUDA(ns_launch_plain(ns_lightning_carry_kernel, grid, dim3(256), 0, d->stream, a));
     }
-    return launch_chunk_kernel<DK, false>(d, a, batch, vec);
+    return launch_chunk_kernel<DK, DV, false, BF16>(d, a, batch, vec);
+}
+
+template <int DV, bool BF16>
+int dispatch_chunked(NsDevice* d, const LightningArgs& a, int batch, int vec)
+{
+    if (a.dim <= 32) return launch_chunked<32, DV, BF16>(d, a, batch, vec);
+    return a.dim <= 64 ? launch_chunked<64, DV, BF16>(d, a, batch, vec) : launch_chunked<128, DV, BF16>(d, a, batch, vec);
 }
 
 }  // namespace
@@ -489,8 +586,8 @@ extern "C" int ns_lightning_chunked(ns_device_t h, uint64_t src, int splits, int
     // Segments when one CTA per (head, sequence, value columns) leaves SMs empty; at least two chunks each.  A source that is one
     // bf16 matrix lies outside the device object's scratch block, which then holds the segments' states.
     const int chunks = (steps + LC - 1) / LC;
-    const int64_t ctas = (int64_t)heads * batch * ((vdim + LDV - 1) / LDV);
-    int64_t segs = segments > 0 ? segments : (2 * d->sm_count) / ctas;
+    const int64_t ctas = (int64_t)heads * batch * (vdim <= 64 ? 1 : (vdim + 127) / 128);
+    int64_t segs = segments > 0 ? segments : (vdim <= 64 ? 2 : 1) * d->sm_count / ctas;
     if (segments == 0 && segs > chunks / 2) segs = chunks / 2;
     if (segs > chunks) segs = chunks;
     if (segs > 1 && src_dtype == NS_BF16) {
@@ -504,7 +601,7 @@ extern "C" int ns_lightning_chunked(ns_device_t h, uint64_t src, int splits, int
         }
     }
     const int vec = ((dim | vdim | q_col | k_col | v_col | src_ld) & 3) == 0 && (src & 15) == 0 && (a.src.slab & 3) == 0;
-    if (dim <= 32) return launch_chunked<32>(d, a, batch, vec);
-    if (dim <= 64) return launch_chunked<64>(d, a, batch, vec);
-    return launch_chunked<128>(d, a, batch, vec);
+    const bool eights = src_dtype == NS_BF16 && ((dim | vdim | q_col | k_col | v_col | src_ld) & 7) == 0 && (src & 15) == 0;
+    if (vdim <= 64) return eights ? dispatch_chunked<64, true>(d, a, batch, vec) : dispatch_chunked<64, false>(d, a, batch, vec);
+    return eights ? dispatch_chunked<128, true>(d, a, batch, vec) : dispatch_chunked<128, false>(d, a, batch, vec);
 }

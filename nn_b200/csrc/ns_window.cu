@@ -121,6 +121,75 @@ __global__ void __launch_bounds__(256) ns_window_append_kernel(const AppendArgs 
     for (int c = tid; c < a.heads * pad; c += 256) ns_store(q + (c / pad) * a.r.k_ld + a.dim + c % pad, 0.0f);
 }
 
+// The same from one bf16 matrix whose columns come in eights (a prompt's portion): Q groups of eight query or key values of a row per
+// thread in registers, values moved as they are.  k_magic, v_magic: group index -> head, head = index * magic >> 32.
+template <int Q>
+__global__ void __launch_bounds__(256) ns_window_append_rows_kernel(const AppendArgs a, uint32_t k_magic, uint32_t v_magic)
+{
+    __shared__ float2 red[8];
+    ns_pdl_wait();
+    ns_pdl_trigger();
+    const int row = blockIdx.x, b = row / a.steps, tid = threadIdx.x;
+    const int slot = a.slots[b], at = (a.pos[slot] + row - b * a.steps) % a.r.ring_len;
+    const uint16_t* src = reinterpret_cast<const uint16_t*>(a.src.ptr) + (int64_t)row * a.src.ld;
+    const int per_k = a.dim / 8, per_v = a.vdim / 8, nq = a.heads * per_k, n = nq + a.kv_heads * per_k, nv = a.kv_heads * per_v;
+    uint4 x[Q];
+    float sq = 0.0f, sk = 0.0f;
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int p = tid + 256 * i;
+        x[i] = make_uint4(0, 0, 0, 0);
+        if (p < n) x[i] = *reinterpret_cast<const uint4*>(src + (p < nq ? a.q_col + p * 8 : a.k_col + (p - nq) * 8));
+    }
+    uint16_t* v = reinterpret_cast<uint16_t*>(a.r.v) + (int64_t)slot * a.r.v_slot_stride + (int64_t)at * a.r.v_ld;
+    for (int p = tid; p < nv; p += 256) {
+        const int head = (int)__umulhi((uint32_t)p, v_magic);
+        *reinterpret_cast<uint4*>(v + (int64_t)head * a.r.ring_len * a.r.v_ld + (p - head * per_v) * 8) = *reinterpret_cast<const uint4*>(src + a.v_col + p * 8);
+    }
+    if (a.gate != nullptr)
+        for (int c = tid; c < a.heads; c += 256) a.gate[(int64_t)row * a.heads + c] = ns_sigmoid(ns_load(src + a.g_col + c));
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const uint32_t w[4] = {x[i].x, x[i].y, x[i].z, x[i].w};
+        float s = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const float lo = __uint_as_float(w[j] << 16), hi = __uint_as_float(w[j] & 0xFFFF0000u);
+            s = fmaf(lo, lo, fmaf(hi, hi, s));
+        }
+        if (tid + 256 * i < nq) sq += s;
+        else sk += s;
+    }
+    sq = ns_warp_sum(sq);
+    sk = ns_warp_sum(sk);
+    if ((tid & 31) == 0) red[tid >> 5] = make_float2(sq, sk);
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) { sq += red[w].x; sk += red[w].y; }
+    const float fq = 1.0f / sqrtf(sq / (float)(nq * 8) + a.eps), fk = 1.0f / sqrtf(sk / (float)((n - nq) * 8) + a.eps);
+    uint16_t* q = reinterpret_cast<uint16_t*>(a.q) + (int64_t)row * a.heads * a.r.k_ld;
+    uint16_t* k = reinterpret_cast<uint16_t*>(a.r.k) + (int64_t)slot * a.r.k_slot_stride + (int64_t)at * a.r.k_ld;
+#pragma unroll
+    for (int i = 0; i < Q; i++) {
+        const int p = tid + 256 * i;
+        if (p >= n) continue;
+        const bool query = p < nq;
+        const int pp = query ? p : p - nq, head = (int)__umulhi((uint32_t)pp, k_magic);
+        const float* w = query ? a.q_norm : a.k_norm;
+        if (w != nullptr) {
+            const float f = query ? fq : fk;
+            const float4 w0 = __ldg(reinterpret_cast<const float4*>(w + pp * 8)), w1 = __ldg(reinterpret_cast<const float4*>(w + pp * 8 + 4));
+            x[i].x = ns_pack_bf16x2(__uint_as_float(x[i].x << 16) * f * w0.x, __uint_as_float(x[i].x & 0xFFFF0000u) * f * w0.y);
+            x[i].y = ns_pack_bf16x2(__uint_as_float(x[i].y << 16) * f * w0.z, __uint_as_float(x[i].y & 0xFFFF0000u) * f * w0.w);
+            x[i].z = ns_pack_bf16x2(__uint_as_float(x[i].z << 16) * f * w1.x, __uint_as_float(x[i].z & 0xFFFF0000u) * f * w1.y);
+            x[i].w = ns_pack_bf16x2(__uint_as_float(x[i].w << 16) * f * w1.z, __uint_as_float(x[i].w & 0xFFFF0000u) * f * w1.w);
+        }
+        uint16_t* dst = query ? q + head * a.r.k_ld : k + (int64_t)head * a.r.ring_len * a.r.k_ld;
+        *reinterpret_cast<uint4*>(dst + (pp - head * per_k) * 8) = x[i];
+    }
+}
+
 // ---------------------------------------------------------------------------------------------
 // 32-bit attention: a warp per (row, head), a lane per key of a block of 32
 // ---------------------------------------------------------------------------------------------
@@ -258,10 +327,10 @@ __global__ void __launch_bounds__(128) ns_window_decode_kernel(const WindowArgs 
 
     auto load_tile = [&](int stage) {
         if (t_load <= t_last) {
-            const int64_t ring_row = (int64_t)t_load * WD_KEYS % a.r.ring_len;
+            const int ring_row = t_load * WD_KEYS % a.r.ring_len;
             const uint32_t sk = mine + stage * L::STAGE * 2, sv = sk + WD_KEYS * L::KLD * 2;
-            const uint16_t* kp = keys + ring_row * k_ld;
-            const uint16_t* vp = values + ring_row * v_ld;
+            const uint16_t* kp = keys + (int64_t)ring_row * k_ld;
+            const uint16_t* vp = values + (int64_t)ring_row * v_ld;
 #pragma unroll
             for (int e = lane; e < WD_KEYS * KS * 2; e += 32) {
                 const int r = e / (KS * 2), c = (e % (KS * 2)) * 8;
@@ -540,6 +609,21 @@ extern "C" int ns_window_append(ns_device_t h, uint64_t src, int splits, int src
     a.steps = steps;
     a.q = reinterpret_cast<void*>(q);
     a.gate = reinterpret_cast<float*>(gate);
+    const int groups = (heads + kv_heads) * (dim / 8);
+    if (dtype == NS_BF16 && src_dtype == NS_BF16 && ((dim | vdim | q_col | k_col | v_col | src_ld) & 7) == 0 && ((src | q_norm | k_norm | q) & 15) == 0 && groups <= 2048 &&
+        kv_heads * (vdim / 8) <= 65535) {
+        // head of a group of eight: index * ceil(2^32 / groups per head) >> 32, exact for indexes and sizes below 2^16 (one group
+        // per head does not fit 32 bits)
+        if (dim > 8 && vdim > 8) {
+            const uint32_t k_magic = (uint32_t)(((1ull << 32) + dim / 8 - 1) / (dim / 8)), v_magic = (uint32_t)(((1ull << 32) + vdim / 8 - 1) / (vdim / 8));
+            auto rows = [&](auto k) -> int {
+                NS_CUDA(ns_launch_plain(k, dim3((unsigned)(batch * steps)), dim3(256), 0, d->stream, a, k_magic, v_magic));
+                return NS_OK;
+            };
+            if (groups <= 512) return rows(ns_window_append_rows_kernel<2>);
+            return groups <= 1024 ? rows(ns_window_append_rows_kernel<4>) : rows(ns_window_append_rows_kernel<8>);
+        }
+    }
     const size_t smem = ((size_t)(heads + kv_heads) * dim + 3) / 4 * 16;
     NS_REQUIRE(smem <= 200 * 1024, NS_ERR_ARGUMENT, "ns_window_append: queries and keys of %zu bytes do not fit shared memory", smem);
     const bool vec = ((dim | vdim | q_col | k_col | v_col | src_ld) & 3) == 0 && ((src | q_norm | k_norm | q) & 15) == 0 && (a.src.slab & 3) == 0;
