@@ -264,18 +264,19 @@ __global__ void __launch_bounds__(128) ns_window_attend_kernel(const WindowArgs 
 }
 
 // ---------------------------------------------------------------------------------------------
-// few tokens, bf16: a CTA per (16 rows, key/value head, sequence, share of the window); each of its four warps walks tiles of 16 keys
-// on its own, with its own maximum, sum and weighted values, and its own copies in flight
+// few tokens, bf16: a CTA per (16 rows, key/value head, sequence, share of the window); each of its warps walks tiles of 16 keys on its
+// own, with its own maximum, sum and weighted values, and its own copies in flight
 // ---------------------------------------------------------------------------------------------
-constexpr int WD_KEYS = 16, WD_STAGES = 3, WD_WARPS = 4;
+constexpr int WD_KEYS = 16, WD_STAGES = 3;
 
-// KS: 16-wide steps over a key; NV: 8-wide column tiles of a value
-template <int KS, int NV>
+// KS: 16-wide steps over a key; NV: 8-wide column tiles of a value; WARPS: 2 where there are several CTAs per SM (short CTAs fill the SMs
+// more evenly: 53 us against 62 for 64 sequences x 16 heads and 512 positions), else 4
+template <int KS, int NV, int WARPS>
 struct DecodeSmem {
     static constexpr int KLD = KS * 16 + 8, VLD = NV * 8 + 8, STAGE = WD_KEYS * (KLD + VLD);       // bf16 elements
     static constexpr int OLD = NV * 8 + 4;                                                         // floats of a row when the warps merge
-    static constexpr int TILES = WD_WARPS * WD_STAGES * STAGE * 2, MERGE = WD_WARPS * 16 * OLD * 4;
-    static constexpr int BYTES = (TILES > MERGE ? TILES : MERGE) + WD_WARPS * 32 * 4;
+    static constexpr int TILES = WARPS * WD_STAGES * STAGE * 2, MERGE = WARPS * 16 * OLD * 4;
+    static constexpr int BYTES = (TILES > MERGE ? TILES : MERGE) + WARPS * 32 * 4;
 };
 
 NS_DEVINL void write_out(const WindowArgs& a, int b, int kvh, int r, int c, float weighted, float f)
@@ -299,10 +300,10 @@ NS_DEVINL float out_factor(const WindowArgs& a, int b, int kvh, int r, float m, 
     return f / l;
 }
 
-template <int KS, int NV>
-__global__ void __launch_bounds__(128) ns_window_decode_kernel(const WindowArgs a)
+template <int KS, int NV, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) ns_window_decode_kernel(const WindowArgs a)
 {
-    using L = DecodeSmem<KS, NV>;
+    using L = DecodeSmem<KS, NV, WARPS>;
     extern __shared__ __align__(16) uint8_t wd_smem[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const uint32_t mine = ns_smem_u32(wd_smem) + warp * WD_STAGES * L::STAGE * 2;
@@ -317,8 +318,8 @@ __global__ void __launch_bounds__(128) ns_window_decode_kernel(const WindowArgs 
     const int last = pos0 + min(row0 + 15, a.rows - 1) / rep, first = max(0, pos0 + row0 / rep - a.window + 1);
     const uint16_t* keys = reinterpret_cast<const uint16_t*>(a.r.k) + (int64_t)slot * a.r.k_slot_stride + (int64_t)kvh * a.r.ring_len * k_ld;
     const uint16_t* values = reinterpret_cast<const uint16_t*>(a.r.v) + (int64_t)slot * a.r.v_slot_stride + (int64_t)kvh * a.r.ring_len * v_ld;
-    const int t_last = last / WD_KEYS, stride = WD_WARPS * a.splits;
-    int t_load = first / WD_KEYS + split * WD_WARPS + warp;
+    const int t_last = last / WD_KEYS, stride = WARPS * a.splits;
+    int t_load = first / WD_KEYS + split * WARPS + warp;
 
     // columns between a row's length and the next multiple of 16 are read: zero in every stage
     if (k_ld < KS * 16)
@@ -439,7 +440,7 @@ __global__ void __launch_bounds__(128) ns_window_decode_kernel(const WindowArgs 
     }
     ns_cp_wait<0>();
 
-    // the four warps' results become one
+    // the warps' results become one
 #pragma unroll
     for (int h = 0; h < 2; h++) {
         l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
@@ -459,12 +460,12 @@ __global__ void __launch_bounds__(128) ns_window_decode_kernel(const WindowArgs 
             *reinterpret_cast<float2*>(sO + (warp * 16 + g + h * 8) * L::OLD + j * 8 + t4 * 2) = make_float2(acc[j][2 * h], acc[j][2 * h + 1]);
     __syncthreads();
     const int count = min(16, a.rows - row0);
-    for (int r = warp; r < count; r += WD_WARPS) {
-        float top = -INFINITY, sum = 0.0f, w[WD_WARPS];
+    for (int r = warp; r < count; r += WARPS) {
+        float top = -INFINITY, sum = 0.0f, w[WARPS];
 #pragma unroll
-        for (int i = 0; i < WD_WARPS; i++) top = fmaxf(top, sM[i * 32 + r]);
+        for (int i = 0; i < WARPS; i++) top = fmaxf(top, sM[i * 32 + r]);
 #pragma unroll
-        for (int i = 0; i < WD_WARPS; i++) {
+        for (int i = 0; i < WARPS; i++) {
             w[i] = top == -INFINITY ? 0.0f : ns_exp2(sM[i * 32 + r] - top);
             sum = fmaf(sM[i * 32 + 16 + r], w[i], sum);
         }
@@ -474,7 +475,7 @@ __global__ void __launch_bounds__(128) ns_window_decode_kernel(const WindowArgs 
         for (int c = lane; c < a.vdim; c += 32) {
             float x = 0.0f;
 #pragma unroll
-            for (int i = 0; i < WD_WARPS; i++) x = fmaf(sO[(i * 16 + r) * L::OLD + c], w[i], x);
+            for (int i = 0; i < WARPS; i++) x = fmaf(sO[(i * 16 + r) * L::OLD + c], w[i], x);
             if (whole) write_out(a, b, kvh, row0 + r, c, x, f);
             else part[c] = x;
         }
@@ -520,15 +521,21 @@ int dispatch_attend(NsDevice* d, const WindowArgs& a, int batch)
     return launch_attend<T, 32>(d, a, batch);
 }
 
+template <int KS, int NV, int WARPS>
+int launch_decode_warps(NsDevice* d, const WindowArgs& a, int batch)
+{
+    constexpr int smem = DecodeSmem<KS, NV, WARPS>::BYTES;
+    static_assert(smem <= 227 * 1024, "a CTA's shared memory");
+    auto k = ns_window_decode_kernel<KS, NV, WARPS>;
+    NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    NS_CUDA(ns_launch_plain(k, dim3((unsigned)((a.rows + 15) / 16 * a.splits), (unsigned)a.kv_heads, (unsigned)batch), dim3(WARPS * 32), (size_t)smem, d->stream, a));
+    return NS_OK;
+}
 template <int KS, int NV>
 int launch_decode(NsDevice* d, const WindowArgs& a, int batch)
 {
-    constexpr int smem = DecodeSmem<KS, NV>::BYTES;
-    static_assert(smem <= 227 * 1024, "a CTA's shared memory");
-    auto k = ns_window_decode_kernel<KS, NV>;
-    NS_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    NS_CUDA(ns_launch_plain(k, dim3((unsigned)((a.rows + 15) / 16 * a.splits), (unsigned)a.kv_heads, (unsigned)batch), dim3(128), (size_t)smem, d->stream, a));
-    return NS_OK;
+    const int64_t ctas = (int64_t)batch * a.kv_heads * ((a.rows + 15) / 16) * a.splits;
+    return ctas >= 4 * (int64_t)d->sm_count ? launch_decode_warps<KS, NV, 2>(d, a, batch) : launch_decode_warps<KS, NV, 4>(d, a, batch);
 }
 template <int KS>
 int dispatch_decode(NsDevice* d, const WindowArgs& a, int batch)
@@ -662,7 +669,7 @@ extern "C" int ns_window_decode(ns_device_t h, uint64_t q, uint64_t k_ring, uint
     const int64_t ctas = (int64_t)batch * kv_heads * ((a.rows + 15) / 16);
     const int tiles = (window - 1 + (steps < 16 ? steps : 16)) / WD_KEYS + 2;
     int64_t splits = 2 * d->sm_count / ctas;
-    if (splits > tiles / (2 * WD_WARPS)) splits = tiles / (2 * WD_WARPS);
+    if (splits > tiles / 8) splits = tiles / 8;
     a.splits = splits < 1 ? 1 : (splits > 32 ? 32 : (int)splits);
     if (a.splits > 1) {
         void* block = nullptr;
