@@ -30,7 +30,7 @@ class TopidraConfig:
     vocab: int
     width: int
     layers: list = field(default_factory=list)
-    eps: float = 1e-6
+    eps: float = 1e-5
     loop: dict | None = None            # start, stop, times
 
     @staticmethod
